@@ -377,8 +377,9 @@ int mtx_engine_rebind_state(mtx_engine* e, const mtx_decode_state* s);
                                h = unit(x) * norm1;  x += mixer(h + conv1(h))  (conv1 as above; with two taps (s, -s) this is the
                                token shift h + (h_prev - h) s);  x += ff(unit(x) * norm2) if the layer has a feed-forward;  then, with
                                a side input, x += unit(side_proj(gelu_tanh(side_gate x) * side_embed[token, side_col ..])) * side_norm.
-                               The embedding output is normed with mtx_layered_config.embed_norm, the final norm uses its weight as
-                               stored.  One mixer per layer: attn or rec (MTX_REC_GDELTA) */
+                               The embedding output is normed with mtx_layered_config.embed_norm (if any), the final norm uses its
+                               weight as stored.  One mixer per layer: attn, latent or rec (MTX_REC_GDELTA); conv1 may be NULL (the mixer
+                               then reads h itself); b_in and bo are added where the projections are */
 
 #define MTX_FF_GELU_GATED 0    /* down(gelu_tanh(gate x) * up x) */
 #define MTX_FF_CLAMPED_GATED 1 /* down(g s(1.702 g) (u + 1)), g = min(gate x, limit), u = clamp(up x, -limit, limit), s = sigmoid */
@@ -421,6 +422,18 @@ typedef struct {
   int32_t pool_shared;     /* 1: the pooled pools belong to the layer whose cache this one reads (same P), which fills them */
   void* kp_pages;          /* [kv_heads, num_pages, pool_slots, dim] */
   void* vp_pages;          /* [kv_heads, num_pages, pool_slots, vdim] */
+  /* -- MTX_NORM_PRE layers, none of them together with pooled blocks, slopes, a cap, head gates or q / k norms -- */
+  int32_t chunk;           /* C > 0 (needs window == 0): positions are cut into chunks of C counted from the sequence's start; a query at
+                              i sees the j <= i with j / C == i / C */
+  int32_t maps;            /* 2: differential attention.  Query head h and key head g hold two vectors each, one per map (projection
+                              rows [q: heads*2*dim | k: kv_heads*2*dim | v: kv_heads*vdim], k_pages [kv_heads*2, ..]: key head g's maps
+                              are pool heads 2g, 2g + 1); both maps are softmaxes of their own over the same values, and with their
+                              results a1, a2 head h's output is diff_scale * unit(a1 - diff_lambda * a2), unit RMS over vdim with the
+                              engine's eps.  0 or 1: one map */
+  float diff_lambda, diff_scale;
+  const float* temp;       /* [heads] or NULL: head h's score is multiplied by temp[h] (before the mixing) */
+  const float* talk;       /* [heads, heads] or NULL: before the softmax score_h becomes sum_g talk[h, g] * score_g.  The key pool is
+                              then [1, num_pages, tokens_per_page, kv_heads*dim]: a token's keys of all key heads side by side */
 } mtx_softmax_attn_desc;
 
 /* Attention through latents (csrc/latent_attention.cuh): queries q = w_uq rmsnorm(dq x) laid out per head as [dim plain | rot_dim
@@ -442,6 +455,8 @@ typedef struct {
   const void* w_uk_t;      /* [heads, kv_rank, dim]: per head, the key expansion transposed */
   const void* w_uv;        /* [heads, vdim, kv_rank] */
   void* pages;             /* [1, num_pages, tokens_per_page, kv_rank + rot_dim] */
+  int32_t window;          /* a query at i sees i - window < j <= i; 0: every j <= i */
+  float rot_amp;           /* multiplies cosine and sine of the rotation (query and key side); 0 = 1 */
 } mtx_latent_attn_desc;
 
 #define MTX_REC_GLA 1   /* S = diag(a) S + k v^T, o = S^T q, a = sigmoid(z)^(1 / tau) per key channel, z = low-rank projection */
@@ -512,6 +527,9 @@ typedef struct {
   int32_t score_softmax;   /* 1: s = softmax(router x) over all experts instead of the sigmoid */
   int32_t plain_weights;   /* 1: the chosen experts' scores are the weights as they are (no renormalisation) */
   int32_t act_silu;        /* 1: an expert is down(silu(gate x) * up x) (no limits) instead of the clamped form */
+  int32_t chosen_softmax;  /* 1: experts are chosen by their logits (+ correction), and the weights are the softmax over the chosen
+                              experts' logits alone (score_softmax / plain_weights are then not read) */
+  const float* router_bias; /* [experts] or NULL: added to the router's logits */
 } mtx_moe_desc;
 
 typedef struct {

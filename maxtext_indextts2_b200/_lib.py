@@ -126,6 +126,9 @@ class SoftmaxAttnDesc(ctypes.Structure):
       + [("softcap", ctypes.c_float)]
       + [(n, ctypes.c_int32) for n in ("norm_whole", "pool", "pool_slots", "pool_shared")]
       + [(n, ctypes.c_void_p) for n in ("kp_pages", "vp_pages")]
+      + [(n, ctypes.c_int32) for n in ("chunk", "maps")]
+      + [(n, ctypes.c_float) for n in ("diff_lambda", "diff_scale")]
+      + [(n, ctypes.c_void_p) for n in ("temp", "talk")]
   )
 
 
@@ -136,6 +139,7 @@ class LatentAttnDesc(ctypes.Structure):
       [(n, ctypes.c_int32) for n in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "rot_half")]
       + [("scale", ctypes.c_float)]
       + [(n, ctypes.c_void_p) for n in ("rot_freq", "q_norm", "kv_norm", "sink", "w_uq", "w_uk_t", "w_uv", "pages")]
+      + [("window", ctypes.c_int32), ("rot_amp", ctypes.c_float)]
   )
 
 
@@ -159,7 +163,8 @@ class MoeDesc(ctypes.Structure):
       [(n, ctypes.c_int32) for n in ("experts", "top", "groups", "keep_groups", "ff", "shared_ff")]
       + [(n, ctypes.c_float) for n in ("limit", "shared_limit")]
       + [(n, ctypes.c_void_p) for n in ("w_router", "correction", "w_gate_up", "w_down", "shared_gate_up", "shared_down")]
-      + [(n, ctypes.c_int32) for n in ("score_softmax", "plain_weights", "act_silu")]
+      + [(n, ctypes.c_int32) for n in ("score_softmax", "plain_weights", "act_silu", "chosen_softmax")]
+      + [("router_bias", ctypes.c_void_p)]
   )
 
 

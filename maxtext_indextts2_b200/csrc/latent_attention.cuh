@@ -36,6 +36,7 @@ struct LatentPrepareArgs {
   const int* page_map;
   int tokens_per_page, max_pages;
   float eps;
+  float rot_amp;          // factor on cosine and sine
 };
 
 template <typename T>
@@ -64,6 +65,8 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentPrepare
     const int c0 = a.rot_half ? i : 2 * i, c1 = a.rot_half ? i + rh : 2 * i + 1;
     float sn, cs;
     rot_sincos(double(p), a.rot_freq[i], &sn, &cs);
+    sn *= a.rot_amp;
+    cs *= a.rot_amp;
     dst[a.kv_rank + c0] = to_act<T>(tail[c0] * cs - tail[c1] * sn);
     dst[a.kv_rank + c1] = to_act<T>(tail[c1] * cs + tail[c0] * sn);
   }
@@ -78,6 +81,7 @@ struct LatentQueryArgs {
   const double* rot_freq;
   const int* pos;
   int heads, dim, rot_dim, kv_rank, rot_half;
+  float rot_amp;         // factor on cosine and sine
 };
 
 template <typename T>
@@ -94,6 +98,8 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const LatentQueryArgs
     T* dst = a.q_full + size_t(r) * H * dl + h * dl + a.kv_rank;
     float sn, cs;
     rot_sincos(dp, a.rot_freq[i], &sn, &cs);
+    sn *= a.rot_amp;
+    cs *= a.rot_amp;
     dst[c0] = to_act<T>(src[c0] * cs - src[c1] * sn);
     dst[c1] = to_act<T>(src[c1] * cs + src[c0] * sn);
   }

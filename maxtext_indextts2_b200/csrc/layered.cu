@@ -2,7 +2,7 @@
 // batches whose keys and values live in page pools.  Host code only: the kernels are in linear_any.cuh (any-shape projections, also
 // grouped by expert), gemm_rows.cuh (the tcgen05 projections, for shapes made of whole 128 x 64 tiles), layer_ops.cuh (norms,
 // residual, cache append), grouped_gemm.cuh (the experts' products of steps with many rows), window_attention*.cuh (the sigmoid window mixer), softmax_attention.cuh (causal softmax attention with
-// rotary positions), recurrent_mixers.cuh (GLA, mLSTM and the delta rule over state slots), latent_attention.cuh (attention through
+// rotary positions), multi_attention.cuh (its tensor-core kernels for two score maps per head and for scores mixed over the heads), recurrent_mixers.cuh (GLA, mLSTM and the delta rule over state slots), latent_attention.cuh (attention through
 // cached latents) and moe.cuh (routing).
 #include <cmath>
 #include <cstdio>
@@ -17,6 +17,7 @@
 #include "window_attention_mma.cuh"
 #include "window_attention_decode.cuh"
 #include "softmax_attention.cuh"
+#include "multi_attention.cuh"
 #include "recurrent_mixers.cuh"
 #include "latent_attention.cuh"
 #include "moe.cuh"
@@ -44,7 +45,8 @@ struct mtx_layered {
   float* attn_part = nullptr;  // fp32 partial outputs of the attention's key splits: room for 4 * max_rows rows
   size_t attn_part_rows = 0;
   float* smax_ml = nullptr;    // the softmax attention's key splits: running maximum and sum per (split, row, head)
-  int max_attn_heads = 0;
+  int max_attn_heads = 0;      // units: query heads x score maps
+  int max_part_cols = 0;       // columns of the partial results of layers with two score maps (float32 engines keep one part of them)
   // composite mixers, sandwich norms, routed feed-forwards
   bool sandwich = false;
   int max_rec_o = 0, max_rec_aux = 0, max_moe_top = 0, max_moe_experts = 0, max_moe_ff = 0;
@@ -93,8 +95,9 @@ LWs layered_layout(const mtx_layered* e) {
   L.act = take(R * (e->max_ff > 0 ? e->max_ff : 1) * es);
   L.wanted = take(W * c.width * es);
   L.obf = take(R * size_t(e->max_nqkv > c.width ? e->max_nqkv : c.width) * 2);  // bf16 output of a tcgen05 projection
-  L.attn_part = take(c.float32 ? 1024 : 4 * R * size_t(e->max_odim) * 4);
-  L.smax_ml = take(c.float32 ? 4 : 4 * R * size_t(e->max_attn_heads > 0 ? e->max_attn_heads : 1) * 2 * 4);
+  const size_t part_cols = size_t(e->max_odim > e->max_part_cols ? e->max_odim : e->max_part_cols);
+  L.attn_part = take(c.float32 ? R * size_t(e->max_part_cols) * 4 + 1024 : 4 * R * part_cols * 4);
+  L.smax_ml = take(c.float32 ? (e->max_part_cols > 0 ? R * size_t(e->max_attn_heads) * 2 * 4 : 4) : 4 * R * size_t(e->max_attn_heads > 0 ? e->max_attn_heads : 1) * 2 * 4);
   L.x0 = take(e->sandwich ? R * c.width * 4 : 4);
   L.rec_o = take(R * size_t(e->max_rec_o > 0 ? e->max_rec_o : 1) * 4);
   L.rec_aux = take(R * size_t(e->max_rec_aux > 0 ? e->max_rec_aux : 1) * 4);
@@ -705,18 +708,96 @@ int launch_softmax_mma_any(const SoftmaxAttnArgs<bf16>& sa, const SoftmaxMmaPlan
   return fail(MTX_ERR_UNSUPPORTED, "no tensor-core attention for dim %d", sa.dim);
 }
 
+template <int DV16, int KT>
+int launch_multi_prefill_t(const SoftmaxAttnArgs<bf16>& sa, const MultiMmaPlan& p, int n_tiles, cudaStream_t st) {
+  static size_t have = 0;  // per instantiation
+  if (p.smem > 48 * 1024 && p.smem > have) {
+    MTX_CUDA(cudaFuncSetAttribute(multi_attention_prefill_kernel<DV16, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(p.smem)));
+    have = p.smem;
+  }
+  return launch(multi_attention_prefill_kernel<DV16, KT>, dim3((n_tiles + p.rt - 1) / p.rt, sa.kv_heads * p.chunks), dim3(kMatThreads), p.smem, st, sa, n_tiles, p.uw,
+                p.rt, p.chunks);
+}
+
+int launch_multi_prefill(const SoftmaxAttnArgs<bf16>& sa, const MultiMmaPlan& p, int n_tiles, cudaStream_t st) {
+  if (p.dv16 == 4 && p.kt == 64) return launch_multi_prefill_t<4, 64>(sa, p, n_tiles, st);
+  if (p.dv16 == 4) return launch_multi_prefill_t<4, 32>(sa, p, n_tiles, st);
+  if (p.dv16 == 8) return launch_multi_prefill_t<8, 32>(sa, p, n_tiles, st);
+  return launch_multi_prefill_t<16, 32>(sa, p, n_tiles, st);
+}
+
+template <int SPW, int DV16>
+int launch_multi_decode_t(const SoftmaxAttnArgs<bf16>& sa, const MultiDecodePlan& p, cudaStream_t st) {
+  static size_t have = 0;  // per instantiation
+  if (p.smem > 48 * 1024 && p.smem > have) {
+    MTX_CUDA(cudaFuncSetAttribute(multi_attention_decode_kernel<SPW, DV16>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(p.smem)));
+    have = p.smem;
+  }
+  return launch(multi_attention_decode_kernel<SPW, DV16>, dim3(sa.rows, p.groups * p.chunks, sa.splits), dim3(128), p.smem, st, sa, p.sets, p.sg, p.chunks);
+}
+
+// key splits as for the other single-token kernel: waves of resident CTAs x (key tiles per split + a split's start-up of two tiles)
+int launch_multi_decode(mtx_layered* e, SoftmaxAttnArgs<bf16>& sa, const MultiDecodePlan& p, cudaStream_t st) {
+  const long long ctas = (long long)sa.rows * p.groups * p.chunks;
+  long long per_sm = (long long)((227 * 1024) / (p.smem + 1024));
+  per_sm = per_sm > 16 ? 16 : (per_sm < 1 ? 1 : per_sm);
+  const long long slots = per_sm * e->num_sms;
+  const int span = sa.window > 0 ? sa.window : (sa.chunk > 0 ? sa.chunk : 2048), kt = 64 / p.sg;
+  const double tiles = double((span + kt - 1) / kt);
+  static const int force = env_int("MTX_SOFTMAX_DECODE_SPLITS", 0);
+  double best = 0.0;
+  sa.splits = 1;
+  for (int sp = 1; sp <= 4; ++sp) {
+    if (size_t(sp) * sa.rows > e->attn_part_rows) break;
+    const double cost = double((ctas * sp + slots - 1) / slots) * (tiles / sp + 2.0);
+    if (sp == 1 || cost < best - 1e-9) {
+      best = cost;
+      sa.splits = sp;
+    }
+  }
+  if (force >= 1 && force <= 4 && size_t(force) * sa.rows <= e->attn_part_rows) sa.splits = force;
+  int rc = MTX_ERR_UNSUPPORTED;
+  if (p.spw == 1 && p.dv16 == 4) rc = launch_multi_decode_t<1, 4>(sa, p, st);
+  else if (p.spw == 1 && p.dv16 == 8) rc = launch_multi_decode_t<1, 8>(sa, p, st);
+  else if (p.spw == 1) rc = launch_multi_decode_t<1, 16>(sa, p, st);
+  else if (p.dv16 == 4) rc = launch_multi_decode_t<2, 4>(sa, p, st);
+  else if (p.dv16 == 8) rc = launch_multi_decode_t<2, 8>(sa, p, st);
+  else rc = launch_multi_decode_t<2, 16>(sa, p, st);
+  MTX_TRY(rc);
+  if (sa.maps > 1) return launch(softmax_diff_merge_kernel<bf16>, dim3((sa.rows * sa.heads + 3) / 4), dim3(128), 0, st, sa);
+  if (sa.splits > 1) return launch(softmax_attention_merge_kernel, dim3((sa.rows * sa.heads + 3) / 4), dim3(128), 0, st, sa);
+  return MTX_OK;
+}
+
 // causal softmax attention of the step's rows over the paged cache: the tensor-core kernels for bf16 engines whose head sizes they
-// are built for (single-token steps: the transposed kernel), else the fp32 row kernel
+// are built for (single-token steps: the transposed kernels), else the fp32 row kernel
 template <typename T>
 int run_softmax_attention(mtx_layered* e, SoftmaxAttnArgs<T>& sa, const mtx_ragged_batch& b, cudaStream_t st) {
-  bool done = false;
+  const int maps = sa.maps > 1 ? sa.maps : 1;
+  const bool multi_shape = maps > 1 || sa.wide;
+  sa.eps = e->cfg.eps;
+  if (multi_shape || sizeof(T) == 2) {
+    sa.part_o = e->attn_part;
+    sa.part_ml = e->smax_ml;
+  }
   if constexpr (sizeof(T) == 2) {
     const SoftmaxMmaPlan plan = softmax_mma_plan(sa.heads, sa.kv_heads, sa.dim, sa.vdim);
     static const int decode_arm = env_int("MTX_SOFTMAX_DECODE", 1);
-    if (plan.ok && use_softmax_mma() && sa.ld_out % 2 == 0) {
-      if (b.n_tiles == sa.rows && decode_arm) MTX_TRY(launch_softmax_decode(e, sa, plan.d16, st));
-      else MTX_TRY(launch_softmax_mma(e, sa, plan, b.n_tiles, b.n_tiles == sa.rows, st));
-      done = true;
+    if (use_softmax_mma() && sa.ld_out % 2 == 0) {
+      if (plan.ok && !multi_shape) {
+        if (b.n_tiles == sa.rows && decode_arm) return launch_softmax_decode(e, sa, plan.d16, st);
+        return launch_softmax_mma(e, sa, plan, b.n_tiles, b.n_tiles == sa.rows, st);
+      }
+      if (sa.pool == 0 && !sa.slopes && sa.softcap == 0.0f) {
+        const bool same_kv = sa.k_pages == sa.v_pages;
+        if (b.n_tiles == sa.rows) {
+          const MultiDecodePlan p = multi_decode_plan(sa.heads, sa.kv_heads, sa.dim, sa.vdim, maps, sa.wide != 0, same_kv);
+          if (p.ok) return launch_multi_decode(e, sa, p, st);
+        } else {
+          const MultiMmaPlan p = multi_mma_plan(sa.heads, sa.kv_heads, sa.dim, sa.vdim, maps, sa.wide != 0, same_kv, b.n_tiles, e->num_sms);
+          if (p.ok) return launch_multi_prefill(sa, p, b.n_tiles, st);
+        }
+      }
     }
   }
   const size_t smem = softmax_attn_smem_bytes(sa.dim, sa.vdim);
@@ -726,7 +807,9 @@ int run_softmax_attention(mtx_layered* e, SoftmaxAttnArgs<T>& sa, const mtx_ragg
     MTX_CUDA(cudaFuncSetAttribute(softmax_attention_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
     have = smem;
   }
-  if (!done) MTX_TRY(launch(softmax_attention_rows_kernel<T>, dim3(b.n_tiles, sa.heads), dim3(kSmaxThreads), smem, st, sa));
+  sa.splits = 1;
+  MTX_TRY(launch(softmax_attention_rows_kernel<T>, dim3(b.n_tiles, sa.heads * maps), dim3(kSmaxThreads), smem, st, sa));
+  if (maps > 1) return launch(softmax_diff_merge_kernel<T>, dim3((sa.rows * sa.heads + 3) / 4), dim3(128), 0, st, sa);
   return MTX_OK;
 }
 
@@ -856,7 +939,7 @@ int composite_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStrea
   if (l.ff_kind == MTX_FF_MOE) {
     const mtx_moe_desc& m = l.moe;
     const int entries = rows * m.top;
-    if (m.experts <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, (const T*)xa, static_cast<const T*>(m.w_router), e->moe_logits, m.experts, E));
+    if (m.experts <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, (const T*)xa, static_cast<const T*>(m.w_router), (const float*)nullptr, e->moe_logits, m.experts, E));
     else MTX_TRY((linear<T, LIN_PLAIN>(e, xa, m.w_router, nullptr, e->moe_logits, nullptr, rows, m.experts, E, st)));
     MoeRouteArgs ra;
     memset(&ra, 0, sizeof(ra));
@@ -985,6 +1068,98 @@ int group_norm_step(mtx_layered* e, const float* y, float mult, int next, const 
   return launch(group_norm_step_kernel<T, false>, grid, dim3(256), 0, st, y, mult, e->x, w, c.eps, e->h, c.width, c.norm_groups, none);
 }
 
+// attention arguments that do not depend on the layer
+template <typename T>
+SoftmaxAttnArgs<T> attention_args(const mtx_layered_config& c, const mtx_ragged_batch& b) {
+  SoftmaxAttnArgs<T> sa;
+  memset(&sa, 0, sizeof(sa));
+  sa.group = b.group;
+  sa.pos = b.pos;
+  sa.page_map = b.page_map;
+  sa.tile_row0 = b.tile_row0;
+  sa.num_pages = c.num_pages;
+  sa.tokens_per_page = c.tokens_per_page;
+  sa.max_pages = c.max_pages_per_group;
+  sa.out_scale = 1.0f;
+  sa.splits = 1;
+  sa.rows = b.rows;
+  return sa;
+}
+
+// a latent attention whose down-projections and head gates lie in the columns q_col, kv_col and g_col of e->qkv [rows, n_in]; the
+// heads go to out [rows, ld_out]
+template <typename T>
+int latent_mixer(mtx_layered* e, const mtx_latent_attn_desc& m, int n_in, int q_col, int kv_col, int g_col, T* out, int ld_out, const mtx_ragged_batch& b,
+                 cudaStream_t st) {
+  const mtx_layered_config& c = e->cfg;
+  const int rows = b.rows;
+  const int H = m.heads, dl = m.kv_rank + m.rot_dim, dq = m.dim + m.rot_dim;
+  T* cq = static_cast<T*>(e->act);        // [rows, q_rank]
+  T* q_plain = static_cast<T*>(e->lat_o);  // [rows, H * dim], consumed before the attention writes its result to the same plane
+  T* q_full = static_cast<T*>(e->q);       // [rows, H * dl]
+  T* o_lat = static_cast<T*>(e->lat_o);    // [rows, H * dl]
+  LatentPrepareArgs<T> la;
+  memset(&la, 0, sizeof(la));
+  la.proj = e->qkv;
+  la.ld = n_in;
+  la.q_col = q_col;
+  la.kv_col = kv_col;
+  la.q_rank = m.q_rank;
+  la.kv_rank = m.kv_rank;
+  la.rot_dim = m.rot_dim;
+  la.rot_half = m.rot_half;
+  la.q_norm = m.q_norm;
+  la.kv_norm = m.kv_norm;
+  la.rot_freq = m.rot_freq;
+  la.cq_out = cq;
+  la.pages = static_cast<T*>(m.pages);
+  la.group = b.group;
+  la.pos = b.pos;
+  la.page_map = b.page_map;
+  la.tokens_per_page = c.tokens_per_page;
+  la.max_pages = c.max_pages_per_group;
+  la.eps = c.eps;
+  la.rot_amp = m.rot_amp != 0.0f ? m.rot_amp : 1.0f;
+  MTX_TRY(launch(latent_prepare_kernel<T>, dim3(rows), dim3(256), 0, st, la));
+  MTX_TRY((linear<T, LIN_PLAIN>(e, cq, m.w_uq, nullptr, e->lat_q, nullptr, rows, H * dq, m.q_rank, st)));
+  LatentQueryArgs<T> lq;
+  memset(&lq, 0, sizeof(lq));
+  lq.q = e->lat_q;
+  lq.q_plain = q_plain;
+  lq.q_full = q_full;
+  lq.rot_freq = m.rot_freq;
+  lq.pos = b.pos;
+  lq.heads = H;
+  lq.dim = m.dim;
+  lq.rot_dim = m.rot_dim;
+  lq.kv_rank = m.kv_rank;
+  lq.rot_half = m.rot_half;
+  lq.rot_amp = la.rot_amp;
+  MTX_TRY(launch(latent_query_kernel<T>, dim3(rows), dim3(256), 0, st, lq));
+  // the plain query parts into the latent space, head by head
+  MTX_TRY(linear_batched<T>(q_plain, (long long)H * m.dim, m.dim, m.w_uk_t, (long long)m.kv_rank * m.dim, q_full, (long long)H * dl, dl, rows, m.kv_rank,
+                            m.dim, H, st));
+  SoftmaxAttnArgs<T> sa = attention_args<T>(c, b);
+  sa.ld_gate = n_in;
+  sa.q = q_full;
+  sa.out = o_lat;
+  sa.ld_out = (long long)H * dl;
+  sa.k_pages = static_cast<const T*>(m.pages);
+  sa.v_pages = static_cast<const T*>(m.pages);  // the values are the cached rows themselves
+  sa.heads = H;
+  sa.kv_heads = 1;
+  sa.dim = dl;
+  sa.vdim = dl;
+  sa.window = m.window;
+  sa.scale = m.scale;
+  sa.sink = m.sink;
+  sa.gate = e->qkv + g_col;
+  MTX_TRY(run_softmax_attention<T>(e, sa, b, st));
+  // ... and the weighted latents out of it
+  MTX_TRY(linear_batched<T>(o_lat, (long long)H * dl, dl, m.w_uv, (long long)m.vdim * m.kv_rank, out, ld_out, m.vdim, rows, m.vdim, m.kv_rank, H, st));
+  return MTX_OK;
+}
+
 // a MTX_NORM_PARALLEL layer; h holds gnorm(x, norm1) on entry
 template <typename T>
 int parallel_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_t st) {
@@ -1003,18 +1178,7 @@ int parallel_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
                      l.conv_taps, (long long)E));
   }
   MTX_TRY((linear<T, LIN_PLAIN>(e, xa, l.w_in, nullptr, e->qkv, nullptr, rows, n_in, E, st)));
-  SoftmaxAttnArgs<T> sa;
-  memset(&sa, 0, sizeof(sa));
-  sa.group = b.group;
-  sa.pos = b.pos;
-  sa.page_map = b.page_map;
-  sa.tile_row0 = b.tile_row0;
-  sa.num_pages = c.num_pages;
-  sa.tokens_per_page = c.tokens_per_page;
-  sa.max_pages = c.max_pages_per_group;
-  sa.out_scale = 1.0f;
-  sa.splits = 1;
-  sa.rows = rows;
+  SoftmaxAttnArgs<T> sa = attention_args<T>(c, b);
   sa.ld_gate = n_in;
   if (l.attn.heads > 0) {
     const mtx_softmax_attn_desc& a = l.attn;
@@ -1062,67 +1226,7 @@ int parallel_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
     sa.gate = a.head_gate ? e->qkv + pc.ag : nullptr;
     MTX_TRY(run_softmax_attention<T>(e, sa, b, st));
   } else if (l.latent.heads > 0) {
-    const mtx_latent_attn_desc& m = l.latent;
-    const int H = m.heads, dl = m.kv_rank + m.rot_dim, dq = m.dim + m.rot_dim;
-    T* cq = static_cast<T*>(e->act);        // [rows, q_rank]
-    T* q_plain = static_cast<T*>(e->lat_o);  // [rows, H * dim], consumed before the attention writes its result to the same plane
-    T* q_full = static_cast<T*>(e->q);       // [rows, H * dl]
-    T* o_lat = static_cast<T*>(e->lat_o);    // [rows, H * dl]
-    LatentPrepareArgs<T> la;
-    memset(&la, 0, sizeof(la));
-    la.proj = e->qkv;
-    la.ld = n_in;
-    la.q_col = pc.lq;
-    la.kv_col = pc.lkv;
-    la.q_rank = m.q_rank;
-    la.kv_rank = m.kv_rank;
-    la.rot_dim = m.rot_dim;
-    la.rot_half = m.rot_half;
-    la.q_norm = m.q_norm;
-    la.kv_norm = m.kv_norm;
-    la.rot_freq = m.rot_freq;
-    la.cq_out = cq;
-    la.pages = static_cast<T*>(m.pages);
-    la.group = b.group;
-    la.pos = b.pos;
-    la.page_map = b.page_map;
-    la.tokens_per_page = c.tokens_per_page;
-    la.max_pages = c.max_pages_per_group;
-    la.eps = c.eps;
-    MTX_TRY(launch(latent_prepare_kernel<T>, dim3(rows), dim3(256), 0, st, la));
-    MTX_TRY((linear<T, LIN_PLAIN>(e, cq, m.w_uq, nullptr, e->lat_q, nullptr, rows, H * dq, m.q_rank, st)));
-    LatentQueryArgs<T> lq;
-    memset(&lq, 0, sizeof(lq));
-    lq.q = e->lat_q;
-    lq.q_plain = q_plain;
-    lq.q_full = q_full;
-    lq.rot_freq = m.rot_freq;
-    lq.pos = b.pos;
-    lq.heads = H;
-    lq.dim = m.dim;
-    lq.rot_dim = m.rot_dim;
-    lq.kv_rank = m.kv_rank;
-    lq.rot_half = m.rot_half;
-    MTX_TRY(launch(latent_query_kernel<T>, dim3(rows), dim3(256), 0, st, lq));
-    // the plain query parts into the latent space, head by head
-    MTX_TRY(linear_batched<T>(q_plain, (long long)H * m.dim, m.dim, m.w_uk_t, (long long)m.kv_rank * m.dim, q_full, (long long)H * dl, dl, rows, m.kv_rank,
-                              m.dim, H, st));
-    sa.q = q_full;
-    sa.out = o_lat;
-    sa.ld_out = (long long)H * dl;
-    sa.k_pages = static_cast<const T*>(m.pages);
-    sa.v_pages = static_cast<const T*>(m.pages);  // the values are the cached rows themselves
-    sa.heads = H;
-    sa.kv_heads = 1;
-    sa.dim = dl;
-    sa.vdim = dl;
-    sa.window = 0;
-    sa.scale = m.scale;
-    sa.sink = m.sink;
-    sa.gate = e->qkv + pc.lg;
-    MTX_TRY(run_softmax_attention<T>(e, sa, b, st));
-    // ... and the weighted latents out of it
-    MTX_TRY(linear_batched<T>(o_lat, (long long)H * dl, dl, m.w_uv, (long long)m.vdim * m.kv_rank, cat, k_cat, m.vdim, rows, m.vdim, m.kv_rank, H, st));
+    MTX_TRY(latent_mixer<T>(e, l.latent, n_in, pc.lq, pc.lkv, pc.lg, cat, k_cat, b, st));
   } else {
     const mtx_recurrent_desc& r = l.rec;
     DeltaPrepareArgs pa;
@@ -1186,6 +1290,7 @@ int parallel_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
 // Column layout of a MTX_NORM_PRE layer's input projection.
 struct PreCols {
   int aq = 0, ak = 0, av = 0;                           // softmax attention: q, k, v
+  int lq = 0, lkv = 0, lg = 0;                          // latent attention: query latent, key / value latent + rotated part, head gates
   int rq = 0, rb = 0, ra = 0, rg = 0;                   // gated delta rule: q | k | v from rq, write strengths, the decay's input, the gate's input
   int n = 0, k_mix = 0;
 };
@@ -1196,15 +1301,25 @@ PreCols pre_cols(const mtx_layer_desc& l) {
   const mtx_recurrent_desc& r = l.rec;
   int at = 0;
   if (a.heads > 0) {
+    const int maps = a.maps > 1 ? a.maps : 1;
     pc.aq = at;
-    at += a.heads * a.dim;
+    at += a.heads * maps * a.dim;
     if (!a.shared_kv) {
       pc.ak = at;
-      at += a.kv_heads * a.dim;
+      at += a.kv_heads * maps * a.dim;
       pc.av = at;
       at += a.kv_heads * a.vdim;
     }
     pc.k_mix = a.heads * a.vdim;
+  } else if (l.latent.heads > 0) {
+    const mtx_latent_attn_desc& m = l.latent;
+    pc.lq = at;
+    at += m.q_rank;
+    pc.lkv = at;
+    at += m.kv_rank + m.rot_dim;
+    pc.lg = at;
+    at += m.heads;
+    pc.k_mix = m.heads * m.vdim;
   } else {
     const int G = r.kv_heads > 0 ? r.kv_heads : r.heads;
     pc.rq = at;
@@ -1223,7 +1338,7 @@ PreCols pre_cols(const mtx_layer_desc& l) {
 
 // MTX_NORM_PRE: x += y (or unit(y) * y_w; y null: no update), optionally a copy of x in the matmul dtype to xb, then unit(x) * w:
 // `next` >= 0: the norm before layer `next`'s mixer (none after the last layer), to the plane h, or -- in steps of single tokens --
-// straight through that layer's input convolution into xa; `next` < 0: the norm `w` before a feed-forward, to xa
+// straight through that layer's input convolution into xa, or -- a layer without one -- to xa; `next` < 0: the norm `w` before a feed-forward, to xa
 template <typename T>
 int pre_norm_step(mtx_layered* e, const float* y, const float* y_w, const float* self_w, bool copy_x, int next, const float* w, const mtx_ragged_batch& b,
                   cudaStream_t st) {
@@ -1245,6 +1360,7 @@ int pre_norm_step(mtx_layered* e, const float* y, const float* y_w, const float*
     }
     const mtx_layer_desc& nl = e->layers[next];
     pa.w = nl.norm1;
+    if (!nl.conv1) return launch(pre_norm_step_kernel<T, false>, dim3(b.rows), dim3(256), 0, st, pa, xc, static_cast<T*>(e->xa), cv);
     if (single_token_rows(b)) {
       cv = input_conv_args<T>(e, nl, b);
       cv.w2 = nullptr;
@@ -1258,7 +1374,8 @@ int pre_norm_step(mtx_layered* e, const float* y, const float* y_w, const float*
   return launch(pre_norm_step_kernel<T, false>, dim3(b.rows), dim3(256), 0, st, pa, xc, static_cast<T*>(e->xa), cv);
 }
 
-// a MTX_NORM_PRE layer; h holds unit(x) * norm1 on entry (steps of single tokens: xa already holds the mixer's input)
+// a MTX_NORM_PRE layer; h holds unit(x) * norm1 on entry (steps of single tokens, and layers without an input convolution: xa
+// already holds the mixer's input)
 template <typename T>
 int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_t st) {
   const mtx_layered_config& c = e->cfg;
@@ -1268,7 +1385,7 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
   const PreCols pc = pre_cols(l);
   const int n_in = l.n_in;
   T* mix = static_cast<T*>(e->attn);  // [rows, k_mix]
-  if (!single_token_rows(b)) {  // (else the kernel that normed the rows has done this too)
+  if (l.conv1 && !single_token_rows(b)) {  // (else the kernel that normed the rows has done this too)
     InputConvArgs<T> ca = input_conv_args<T>(e, l, b);
     ca.w2 = nullptr;
     ca.out2 = nullptr;
@@ -1277,7 +1394,8 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
       MTX_TRY(launch(conv_state_update_kernel, dim3(b.n_runs, l.conv_taps - 1), dim3(256), 0, st, (const float*)e->h, l.conv_state, b.run_row0, b.group, b.pos, E,
                      l.conv_taps, (long long)E));
   }
-  MTX_TRY((linear<T, LIN_PLAIN>(e, xa, l.w_in, nullptr, e->qkv, nullptr, rows, n_in, E, st)));
+  if (l.b_in) MTX_TRY((linear<T, LIN_BIAS>(e, xa, l.w_in, l.b_in, e->qkv, nullptr, rows, n_in, E, st)));
+  else MTX_TRY((linear<T, LIN_PLAIN>(e, xa, l.w_in, nullptr, e->qkv, nullptr, rows, n_in, E, st)));
   if (l.attn.heads > 0) {
     const mtx_softmax_attn_desc& a = l.attn;
     QkPrepareArgs<T> qa;
@@ -1308,7 +1426,12 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
     qa.tokens_per_page = c.tokens_per_page;
     qa.max_pages = c.max_pages_per_group;
     qa.eps = c.eps;
-    MTX_TRY(launch(qk_prepare_append_kernel<T>, dim3(rows), dim3(256), 0, st, qa));
+    qa.maps = a.maps;
+    qa.temp = a.temp;
+    qa.talk = a.talk;
+    const size_t qsmem = a.talk ? sizeof(float) * a.heads * a.dim : 0;
+    if (qsmem > 48 * 1024) MTX_CUDA(cudaFuncSetAttribute(qk_prepare_append_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(qsmem)));
+    MTX_TRY(launch(qk_prepare_append_kernel<T>, dim3(rows), dim3(256), qsmem, st, qa));
     if (a.pool > 0 && !a.pool_shared) {  // the blocks that this step's rows complete
       PoolAppendArgs<T> pa;
       memset(&pa, 0, sizeof(pa));
@@ -1329,18 +1452,8 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
       pa.max_pages = c.max_pages_per_group;
       MTX_TRY(launch(pool_append_kernel<T>, dim3(rows), dim3(256), 0, st, pa));
     }
-    SoftmaxAttnArgs<T> sa;
-    memset(&sa, 0, sizeof(sa));
-    sa.group = b.group;
-    sa.pos = b.pos;
-    sa.page_map = b.page_map;
-    sa.tile_row0 = b.tile_row0;
-    sa.num_pages = c.num_pages;
-    sa.tokens_per_page = c.tokens_per_page;
-    sa.max_pages = c.max_pages_per_group;
+    SoftmaxAttnArgs<T> sa = attention_args<T>(c, b);
     sa.out_scale = a.out_scale != 0.0f ? a.out_scale : 1.0f;
-    sa.splits = 1;
-    sa.rows = rows;
     sa.q = static_cast<const T*>(e->q);
     sa.out = mix;
     sa.ld_out = pc.k_mix;
@@ -1348,9 +1461,14 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
     sa.v_pages = static_cast<const T*>(a.v_pages);
     sa.heads = a.heads;
     sa.kv_heads = a.kv_heads;
-    sa.dim = a.dim;
+    sa.dim = a.talk ? a.kv_heads * a.dim : a.dim;
     sa.vdim = a.vdim;
     sa.window = a.window;
+    sa.chunk = a.chunk;
+    sa.maps = a.maps;
+    sa.wide = a.talk ? 1 : 0;
+    sa.diff_lambda = a.diff_lambda;
+    sa.diff_scale = a.diff_scale;
     sa.scale = a.scale;
     sa.slopes = a.slopes;
     sa.sink = a.sink;
@@ -1360,6 +1478,8 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
     sa.kp_pages = static_cast<const T*>(a.kp_pages);
     sa.vp_pages = static_cast<const T*>(a.vp_pages);
     MTX_TRY(run_softmax_attention<T>(e, sa, b, st));
+  } else if (l.latent.heads > 0) {
+    MTX_TRY(latent_mixer<T>(e, l.latent, n_in, pc.lq, pc.lkv, pc.lg, mix, pc.k_mix, b, st));
   } else {
     const mtx_recurrent_desc& r = l.rec;
     const int G = r.kv_heads > 0 ? r.kv_heads : r.heads, C = 2 * G * r.dim + r.heads * r.vdim;
@@ -1450,15 +1570,18 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
     oa.out_scale = r.out_scale != 0.0f ? r.out_scale : 1.0f;
     MTX_TRY(launch(recurrent_out_kernel<T>, dim3(rows), dim3(256), 0, st, oa));
   }
-  MTX_TRY((linear<T, LIN_PLAIN>(e, mix, l.wo, nullptr, e->y, nullptr, rows, E, pc.k_mix, st)));
+  if (l.bo) MTX_TRY((linear<T, LIN_BIAS>(e, mix, l.wo, l.bo, e->y, nullptr, rows, E, pc.k_mix, st)));
+  else MTX_TRY((linear<T, LIN_PLAIN>(e, mix, l.wo, nullptr, e->y, nullptr, rows, E, pc.k_mix, st)));
   const mtx_moe_desc& m = l.moe;
   const bool has_ff = m.experts > 0, has_side = l.side_dim > 0;
   if (has_ff) {
     MTX_TRY(pre_norm_step<T>(e, e->y, nullptr, nullptr, false, -1, l.norm2, b, st));  // x += mixer; xa = unit(x) * norm2
     const int entries = rows * m.top;
     const float limit = m.act_silu ? 0.0f : m.limit, shared_limit = m.act_silu ? 0.0f : m.shared_limit;
-    if (m.experts <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, (const T*)xa, static_cast<const T*>(m.w_router), e->moe_logits, m.experts, E));
-    else MTX_TRY((linear<T, LIN_PLAIN>(e, xa, m.w_router, nullptr, e->moe_logits, nullptr, rows, m.experts, E, st)));
+    if (m.experts <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, (const T*)xa, static_cast<const T*>(m.w_router), m.router_bias, e->moe_logits, m.experts, E));
+    // (more experts: the any-shape kernel, whose result is fp32; the tcgen05 projection would round it)
+    else if (m.router_bias) MTX_TRY((run_linear<T, LIN_BIAS>(e, xa, m.w_router, m.router_bias, e->moe_logits, nullptr, rows, m.experts, E, st)));
+    else MTX_TRY((run_linear<T, LIN_PLAIN>(e, xa, m.w_router, nullptr, e->moe_logits, nullptr, rows, m.experts, E, st)));
     MoeRouteArgs ra;
     memset(&ra, 0, sizeof(ra));
     ra.logits = e->moe_logits;
@@ -1471,6 +1594,7 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
     ra.keep = m.keep_groups > 0 ? m.keep_groups : 1;
     ra.softmax = m.score_softmax;
     ra.plain = m.plain_weights;
+    ra.chosen_softmax = m.chosen_softmax;
     MTX_TRY(launch(moe_route_kernel, dim3(rows), dim3(32), sizeof(float) * (2 * m.experts + ra.groups), st, ra));
     MTX_TRY(launch(moe_sort_kernel, dim3(1), dim3(1024), sizeof(int) * (2 * m.experts + 1), st, (const int*)e->moe_chosen, entries, m.top, m.experts,
                    e->moe_off, e->moe_slot, e->moe_row));
@@ -1590,6 +1714,27 @@ int check_composite(mtx_layered* e, int i) {
   return MTX_OK;
 }
 
+// validation and workspace sizes of a layer's latent attention
+int check_latent(mtx_layered* e, int i) {
+  const mtx_latent_attn_desc& m = e->layers[i].latent;
+  if (m.dim < 1 || m.rot_dim < 0 || m.vdim < 1 || m.q_rank < 1 || m.kv_rank < 1) return fail(MTX_ERR_ARG, "layer %d: bad latent attention geometry", i);
+  if (m.rot_dim > 0 && !m.rot_freq) return fail(MTX_ERR_ARG, "layer %d: rot_freq is missing", i);
+  if (!m.q_norm || !m.kv_norm || !m.w_uq || !m.w_uk_t || !m.w_uv || !m.pages) return fail(MTX_ERR_ARG, "layer %d: a latent attention weight or its pool is missing", i);
+  const int dl = m.kv_rank + m.rot_dim;
+  if (kSmaxRows * dl > kSmaxThreads * kSmaxMaxAcc) return fail(MTX_ERR_UNSUPPORTED, "layer %d: kv_rank + rot_dim = %d exceeds %d", i, dl, kSmaxThreads * kSmaxMaxAcc / kSmaxRows);
+  if (softmax_attn_smem_bytes(dl, dl) > 200 * 1024) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the latent rows do not fit shared memory", i);
+  if (m.heads * dl > e->max_qdim) e->max_qdim = m.heads * dl;
+  if (m.heads * dl > e->max_lat_o) e->max_lat_o = m.heads * dl;
+  if (m.heads * dl > e->max_odim) e->max_odim = m.heads * dl;  // (the key splits' partial results are sized by max_odim)
+  if (m.heads * m.dim > e->max_lat_o) e->max_lat_o = m.heads * m.dim;
+  if (m.heads * (m.dim + m.rot_dim) > e->max_lat_q) e->max_lat_q = m.heads * (m.dim + m.rot_dim);
+  if (m.q_rank > e->max_ff) e->max_ff = m.q_rank;  // (the query latent waits in the plane of the feed-forward's activation)
+  if (m.heads > e->max_attn_heads) e->max_attn_heads = m.heads;
+  if (m.window < 0) return fail(MTX_ERR_ARG, "layer %d: window", i);
+  if (m.heads * (m.dim + m.rot_dim) > e->max_nqkv) e->max_nqkv = m.heads * (m.dim + m.rot_dim);  // (a tcgen05 projection parks its bf16 result there)
+  return MTX_OK;
+}
+
 // validation and workspace sizes of a MTX_NORM_PARALLEL layer
 int check_parallel(mtx_layered* e, int i) {
   const mtx_layered_config& c = e->cfg;
@@ -1614,19 +1759,7 @@ int check_parallel(mtx_layered* e, int i) {
     if (a.heads > e->max_attn_heads) e->max_attn_heads = a.heads;
   }
   if (m.heads > 0) {
-    if (m.dim < 1 || m.rot_dim < 0 || m.vdim < 1 || m.q_rank < 1 || m.kv_rank < 1) return fail(MTX_ERR_ARG, "layer %d: bad latent attention geometry", i);
-    if (m.rot_dim > 0 && !m.rot_freq) return fail(MTX_ERR_ARG, "layer %d: rot_freq is missing", i);
-    if (!m.q_norm || !m.kv_norm || !m.w_uq || !m.w_uk_t || !m.w_uv || !m.pages) return fail(MTX_ERR_ARG, "layer %d: a latent attention weight or its pool is missing", i);
-    const int dl = m.kv_rank + m.rot_dim;
-    if (kSmaxRows * dl > kSmaxThreads * kSmaxMaxAcc) return fail(MTX_ERR_UNSUPPORTED, "layer %d: kv_rank + rot_dim = %d exceeds %d", i, dl, kSmaxThreads * kSmaxMaxAcc / kSmaxRows);
-    if (softmax_attn_smem_bytes(dl, dl) > 200 * 1024) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the latent rows do not fit shared memory", i);
-    if (m.heads * dl > e->max_qdim) e->max_qdim = m.heads * dl;
-    if (m.heads * dl > e->max_lat_o) e->max_lat_o = m.heads * dl;
-    if (m.heads * dl > e->max_odim) e->max_odim = m.heads * dl;  // (the key splits' partial results are sized by max_odim)
-    if (m.heads * m.dim > e->max_lat_o) e->max_lat_o = m.heads * m.dim;
-    if (m.heads * (m.dim + m.rot_dim) > e->max_lat_q) e->max_lat_q = m.heads * (m.dim + m.rot_dim);
-    if (m.q_rank > e->max_ff) e->max_ff = m.q_rank;  // (the query latent waits in the plane of the feed-forward's activation)
-    if (m.heads > e->max_attn_heads) e->max_attn_heads = m.heads;
+    MTX_TRY(check_latent(e, i));
   }
   if (r.kind != 0) {
     if (r.kind != MTX_REC_DELTA) return fail(MTX_ERR_UNSUPPORTED, "layer %d: a parallel layer's recurrence is the delta rule", i);
@@ -1641,7 +1774,6 @@ int check_parallel(mtx_layered* e, int i) {
   if (l.ff < 0 || (l.ff > 0 && (l.ff_kind != MTX_FF_RELU2 || !l.w_gate_up))) return fail(MTX_ERR_ARG, "layer %d: a parallel layer's feed-forward is down(relu(up x)^2)", i);
   if (pc.k_mix + l.ff > e->max_odim) e->max_odim = pc.k_mix + l.ff;
   if (l.ff > e->max_nqkv) e->max_nqkv = l.ff;  // (a tcgen05 projection parks its bf16 result in a plane of max_nqkv columns)
-  if (m.heads > 0 && m.heads * (m.dim + m.rot_dim) > e->max_nqkv) e->max_nqkv = m.heads * (m.dim + m.rot_dim);
   e->parallel = true;
   return MTX_OK;
 }
@@ -1655,8 +1787,8 @@ int check_prenorm(mtx_layered* e, int i) {
   const mtx_moe_desc& m = l.moe;
   if (l.mixer != MTX_MIXER_COMPOSITE) return fail(MTX_ERR_UNSUPPORTED, "layer %d: a pre-norm layer has a composite mixer", i);
   if (!l.norm1 || !l.w_in || !l.wo) return fail(MTX_ERR_ARG, "layer %d: the norm weight or a projection is missing", i);
-  if (l.conv_taps < 1 || !l.conv1 || (l.conv_taps > 1 && !l.conv_state)) return fail(MTX_ERR_ARG, "layer %d: the input convolution's taps / weights / state", i);
-  if ((a.heads > 0) + (r.kind != 0) != 1 || l.latent.heads > 0) return fail(MTX_ERR_ARG, "layer %d: a pre-norm layer has one mixer, an attention or a recurrence", i);
+  if (l.conv1 ? l.conv_taps < 1 || (l.conv_taps > 1 && !l.conv_state) : l.conv_taps > 1) return fail(MTX_ERR_ARG, "layer %d: the input convolution's taps / weights / state", i);
+  if ((a.heads > 0) + (l.latent.heads > 0) + (r.kind != 0) != 1) return fail(MTX_ERR_ARG, "layer %d: a pre-norm layer has one mixer, an attention, a latent attention or a recurrence", i);
   if (a.heads > 0) {
     if (a.kv_heads < 1 || a.heads % a.kv_heads != 0 || a.dim < 1 || a.vdim < 1 || a.window < 0) return fail(MTX_ERR_ARG, "layer %d: bad attention geometry", i);
     if (a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims & 1) || (a.rot_dims > 0 && !a.rot_freq)) return fail(MTX_ERR_ARG, "layer %d: bad rot_dims / rot_freq", i);
@@ -1667,9 +1799,19 @@ int check_prenorm(mtx_layered* e, int i) {
     if (a.pool > 0 && !(c.tokens_per_page % a.pool == 0 ? a.pool_slots == c.tokens_per_page / a.pool : a.pool_slots == c.tokens_per_page))
       return fail(MTX_ERR_ARG, "layer %d: pool_slots = %d does not fit pages of %d tokens and blocks of %d", i, a.pool_slots, c.tokens_per_page, a.pool);
     if (kSmaxRows * a.vdim > kSmaxThreads * kSmaxMaxAcc) return fail(MTX_ERR_UNSUPPORTED, "layer %d: vdim %d exceeds %d", i, a.vdim, kSmaxThreads * kSmaxMaxAcc / kSmaxRows);
-    if (softmax_attn_smem_bytes(a.dim, a.vdim) > 200 * 1024) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the attention's heads do not fit shared memory", i);
-    if (a.heads * a.dim > e->max_qdim) e->max_qdim = a.heads * a.dim;
-    if (a.heads > e->max_attn_heads) e->max_attn_heads = a.heads;
+    const int maps = a.maps > 1 ? a.maps : 1;
+    if (maps > 2 || a.chunk < 0 || (a.chunk > 0 && a.window > 0) || (maps == 2 && a.talk)) return fail(MTX_ERR_ARG, "layer %d: maps / chunk / talk", i);
+    if ((maps == 2 || a.talk || a.chunk > 0) && (a.pool > 0 || a.slopes || a.softcap > 0.0f || a.q_norm || a.k_norm))
+      return fail(MTX_ERR_UNSUPPORTED, "layer %d: two maps, mixed scores and chunks do not go together with pooled blocks, slopes, a cap or q / k norms", i);
+    if (maps == 2 && a.sink) return fail(MTX_ERR_UNSUPPORTED, "layer %d: a differential attention has no sink", i);
+    if (a.talk && sizeof(float) * a.heads * a.dim > 200 * 1024) return fail(MTX_ERR_UNSUPPORTED, "layer %d: heads * dim = %d of mixed queries", i, a.heads * a.dim);
+    if (softmax_attn_smem_bytes(a.talk ? a.kv_heads * a.dim : a.dim, a.vdim) > 200 * 1024) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the attention's heads do not fit shared memory", i);
+    const int qdim = a.heads * a.dim * (a.talk ? a.kv_heads : maps);
+    if (qdim > e->max_qdim) e->max_qdim = qdim;
+    if (a.heads * maps > e->max_attn_heads) e->max_attn_heads = a.heads * maps;
+    if (maps == 2 && a.heads * maps * a.vdim > e->max_part_cols) e->max_part_cols = a.heads * maps * a.vdim;
+  } else if (l.latent.heads > 0) {
+    MTX_TRY(check_latent(e, i));
   } else {
     if (r.kind != MTX_REC_GDELTA) return fail(MTX_ERR_UNSUPPORTED, "layer %d: a pre-norm layer's recurrence is the gated delta rule", i);
     const int G = r.kv_heads > 0 ? r.kv_heads : r.heads;

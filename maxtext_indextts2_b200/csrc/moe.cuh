@@ -1,10 +1,11 @@
 // Routing of a mixture of experts for a ragged batch (the experts' matrix products are the grouped mode of linear_any.cuh).
 //
-//   moe_router_kernel   per row: the router's logits, fp32 accumulation
+//   moe_router_kernel   per row: the router's logits (plus a bias), fp32 accumulation
 //   moe_route_kernel    per row: s = sigmoid(logits) (or, softmax set, the softmax over all experts); choice = s + correction; the experts of all but the keep_groups best groups
 //                       (a group's score = the sum of its two largest choice scores) are barred; the `top` largest remaining choice
 //                       scores are chosen (the lower index wins a tie); weights = s of the chosen / (their sum + 1e-20), or, plain set, s of the
-//                       chosen as it is.  fp32.
+//                       chosen as it is.  With chosen_softmax the experts are chosen by logit + correction and
+//                       the weights are the softmax over the chosen experts' logits.  fp32.
 //   moe_sort_kernel     one CTA: counts the (row, choice) entries per expert, lays the experts' slot ranges side by side
 //                       (group_off), gives every entry a slot in its expert's range and records the row each slot reads.
 //   moe_combine_kernel  y[row] (+)= sum over the row's choices, in the order of the choices, of weight * expert output of its slot.
@@ -18,7 +19,7 @@ namespace mtx {
 // logits[r, e] = <x[r, :], w[e, :]> with fp32 accumulation: one CTA per row, a warp per expert in turn (few experts, so a tile of
 // a matrix-product kernel would be mostly padding and its k loop one long chain)
 template <typename T>
-__global__ void __launch_bounds__(256) moe_router_kernel(const T* x, const T* w, float* logits, int experts, int width) {
+__global__ void __launch_bounds__(256) moe_router_kernel(const T* x, const T* w, const float* bias, float* logits, int experts, int width) {
   griddep_wait();
   const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* xr = x + size_t(r) * width;
@@ -48,7 +49,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const T* x, const T* w,
       if (c < width) acc0 = fmaf(act_f32(xr[c]), act_f32(we[c]), acc0);
     }
     const float sum = warp_sum(acc0 + acc1);
-    if (lane == 0) logits[size_t(r) * experts + e] = sum;
+    if (lane == 0) logits[size_t(r) * experts + e] = bias ? sum + bias[e] : sum;
   }
 }
 
@@ -60,6 +61,7 @@ struct MoeRouteArgs {
   int experts, top, groups, keep;
   int softmax;              // 1: s = softmax(logits) over all experts
   int plain;                // 1: weights = s of the chosen, not renormalised
+  int chosen_softmax;       // 1: s = logits; weights = softmax over the chosen
 };
 
 // one warp per row; shared memory: 2 * experts + groups floats
@@ -81,7 +83,7 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const MoeRouteArgs a) {
   }
   for (int e = lane; e < E; e += 32) {
     const float z = a.logits[size_t(r) * E + e];
-    const float v = a.softmax ? expf(z - zmax) / zsum : 1.0f / (1.0f + expf(-z));
+    const float v = a.chosen_softmax ? z : a.softmax ? expf(z - zmax) / zsum : 1.0f / (1.0f + expf(-z));
     s[e] = v;
     c[e] = v + (a.correction ? a.correction[e] : 0.0f);
   }
@@ -109,7 +111,7 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const MoeRouteArgs a) {
     }
     __syncwarp();
   }
-  float total = 0.0f;
+  float total = 0.0f, zbest = -INFINITY;
   for (int k = 0; k < a.top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -129,11 +131,19 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const MoeRouteArgs a) {
     }
     if (at == 0x7fffffff) at = 0;  // (fewer admissible experts than `top`: cannot happen for a valid config)
     total += s[at];
+    zbest = fmaxf(zbest, s[at]);
     if (lane == 0) {
       a.chosen[size_t(r) * a.top + k] = at;
       c[at] = -INFINITY;
     }
     __syncwarp();
+  }
+  if (a.chosen_softmax) {
+    float part = 0.0f;
+    for (int k = lane; k < a.top; k += 32) part += expf(s[a.chosen[size_t(r) * a.top + k]] - zbest);
+    const float sum = warp_sum(part);
+    for (int k = lane; k < a.top; k += 32) a.weight[size_t(r) * a.top + k] = expf(s[a.chosen[size_t(r) * a.top + k]] - zbest) / sum;
+    return;
   }
   for (int k = lane; k < a.top; k += 32) a.weight[size_t(r) * a.top + k] = s[a.chosen[size_t(r) * a.top + k]] / (a.plain ? 1.0f : total + 1e-20f);
 }

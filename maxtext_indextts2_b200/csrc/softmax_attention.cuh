@@ -20,6 +20,17 @@
 // the same softmax.  The means live in pools of their own with pool_slots blocks per page, on the sequence's page map (block b in
 // page b / pool_slots), and the kernels walk them as a first segment of keys before the window's tokens.
 //
+// A chunk size instead of a window (chunk > 0): a query at i sees the keys j <= i of its own chunk, j / chunk == i / chunk.
+//
+// Two optional shapes of the scores (multi_attention.cuh has their tensor-core kernels):
+//   * maps == 2: every query head and every key head holds two vectors (score maps) over the same values; unit u = 2 h + m is
+//     head h's map m and reads key head 2 g + m, value head g.  The units' unnormalised results go to part_o / part_ml, and
+//     softmax_diff_merge_kernel takes the maps' difference.
+//   * wide == 1: the heads' scores are mixed before the softmax, score_h = sum_g talk[h, g] <q_g, k_{g's head}>.  The sum over g is taken
+//     on the query's side: qk_prepare_append_kernel writes, per head h, the mixed query (for every key head c the vector
+//     sum over c's query heads g of talk[h, g] q_g), and a token's keys of all key heads are one cached row, so that the score is one
+//     product over kv_heads * d channels (`dim` below) and everything after it is a plain softmax attention.
+//
 //   rope_append_kernel         per row: bias already in the projection; rotates q and k, writes q, appends k and v to the pages
 //   qk_prepare_append_kernel   the same with the optional head norms, either pairing, and layers that append nothing
 //   pool_append_kernel         per row that completes a block: the means of the block's cached keys and values into the pooled pools
@@ -125,6 +136,10 @@ struct QkPrepareArgs {
   int num_pages, tokens_per_page, max_pages;
   float eps;
   int norm_whole;        // 1: q_norm [H * d] / k_norm [G * d]: the whole projection is brought to unit RMS at once
+  int maps;              // 2: heads and key heads hold two vectors each (heads / kv_heads count pairs); else one
+  const float* temp;     // [H]: query head h is multiplied by temp[h] (as its scores would be), or null
+  const float* talk;     // [H, H]: q_out is [rows, H, G * d], the mixed queries, and k_pages holds rows of G * d channels; or null.
+                         // Shared memory: H * d floats
 };
 
 // angle of channel pair c at position p, reduced to [-pi, pi] in double before the fp32 sine and cosine
@@ -138,11 +153,15 @@ template <typename T>
 __global__ void __launch_bounds__(256) qk_prepare_append_kernel(const QkPrepareArgs<T> a) {
   griddep_wait();
   const int r = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
-  const int H = a.heads, G = a.shared_kv ? 0 : a.kv_heads, d = a.dim, dv = a.vdim, rh = a.rot_dims / 2;
+  extern __shared__ float qkp_rows[];  // talk: the row's rotated queries
+  const int maps = a.maps > 1 ? a.maps : 1;
+  const int H = a.heads * maps, G = a.shared_kv ? 0 : a.kv_heads * maps, d = a.dim, dv = a.vdim, rh = a.rot_dims / 2;
   const float* row = a.proj + size_t(r) * a.ld;
   const int p = a.pos[r], grp = a.group[r];
   const size_t slot = size_t(a.page_map[size_t(grp) * a.max_pages + p / a.tokens_per_page]) * a.tokens_per_page + p % a.tokens_per_page;
   const double dp = double(p);
+  // a key head's vectors: rows of its own pool, or (talk) a part of the token's one row
+  const size_t k_head = a.talk ? size_t(d) : size_t(a.num_pages) * a.tokens_per_page * d, k_slot = slot * (a.talk ? size_t(a.kv_heads) * d : size_t(d));
   float inv_all[2] = {1.0f, 1.0f};  // norm_whole: of the query / the key projection
   if (a.norm_whole) {
     __shared__ float red[8];
@@ -169,20 +188,40 @@ __global__ void __launch_bounds__(256) qk_prepare_append_kernel(const QkPrepareA
       ss = warp_sum(ss);
       inv = 1.0f / sqrtf(ss / float(d) + a.eps);
     }
-    T* dst = is_q ? a.q_out + size_t(r) * H * d + u * d : a.k_pages + (size_t(u - H) * a.num_pages * a.tokens_per_page + slot) * d;
-    auto val = [&](int c) { return w ? src[c] * inv * w[c] : src[c]; };
+    T* dst = is_q ? a.q_out + size_t(r) * H * d + u * d : a.k_pages + size_t(u - H) * k_head + k_slot;
+    const float tm = (is_q && a.temp) ? a.temp[u / maps] : 1.0f;
+    auto val = [&](int c) { return (w ? src[c] * inv * w[c] : src[c]) * tm; };
+    auto put = [&](int c, float v) {
+      if (is_q && a.talk) qkp_rows[u * d + c] = v;
+      else dst[c] = to_act<T>(v);
+    };
     for (int i = lane; i < rh; i += 32) {  // the pairs that turn
       const int c0 = a.rot_half ? i : 2 * i, c1 = a.rot_half ? i + rh : 2 * i + 1;
       float sn, cs;
       rot_sincos(dp, a.rot_freq[i], &sn, &cs);
       const float x0 = val(c0), x1 = val(c1);
-      dst[c0] = to_act<T>(x0 * cs - x1 * sn);
-      dst[c1] = to_act<T>(x1 * cs + x0 * sn);
+      put(c0, x0 * cs - x1 * sn);
+      put(c1, x1 * cs + x0 * sn);
     }
-    for (int c = 2 * rh + lane; c < d; c += 32) dst[c] = to_act<T>(val(c));
+    for (int c = 2 * rh + lane; c < d; c += 32) put(c, val(c));
+  }
+  if (a.talk) {  // mixed queries: a thread keeps one channel of one key head's queries and writes it for every head
+    __syncthreads();
+    const int kvh = a.kv_heads, rep = H / kvh, kd = kvh * d;
+    for (int e = tid; e < kd; e += blockDim.x) {
+      const int kv = e / d, c = e % d;
+      const float* sq = qkp_rows + kv * rep * d + c;
+      T* out = a.q_out + size_t(r) * H * kd + e;
+      for (int h = 0; h < H; ++h) {
+        const float* th = a.talk + h * H + kv * rep;
+        float m = 0.0f;
+        for (int g = 0; g < rep; ++g) m = fmaf(th[g], sq[g * d], m);
+        out[size_t(h) * kd] = to_act<T>(m);
+      }
+    }
   }
   if (a.shared_kv) return;
-  for (int e = tid; e < G * dv; e += blockDim.x) {
+  for (int e = tid; e < a.kv_heads * dv; e += blockDim.x) {
     const int kv = e / dv, c = e % dv;
     a.v_pages[(size_t(kv) * a.num_pages * a.tokens_per_page + slot) * dv + c] = to_act<T>(row[a.v_col + e]);
   }
@@ -254,7 +293,16 @@ struct SoftmaxAttnArgs {
   int pool, pool_slots; // pool > 0: pooled blocks (see the head of this file); needs window > 0
   const T* kp_pages;    // [G, num_pages, pool_slots, d]
   const T* vp_pages;    // [G, num_pages, pool_slots, dv]
+  int chunk;            // > 0 (window == 0): a query sees its own chunk of `chunk` positions up to itself
+  int maps, wide;       // see the head of this file (0: one map per head, a key head per value head)
+  float diff_lambda, diff_scale, eps;  // maps == 2
 };
+
+// the first position that the query at position i sees
+__device__ __forceinline__ int smax_first(int i, int window, int chunk) {
+  if (chunk > 0) return i - i % chunk;
+  return window > 0 && i - window + 1 > 0 ? i - window + 1 : 0;
+}
 
 // blocks of `pool` tokens that the query at position i sees: those that end at or before i - window
 __device__ __forceinline__ int smax_blocks_seen(int i, int window, int pool) {
@@ -285,7 +333,9 @@ __device__ __forceinline__ float smax_gate(const float* gate, long long ld, int 
 constexpr int kSmaxThreads = 256, kSmaxRows = 16, kSmaxKeys = 32;
 constexpr int kSmaxMaxAcc = 32;  // kSmaxRows * vdim <= kSmaxThreads * kSmaxMaxAcc: vdim <= 512
 
+constexpr int kSmaxSlice = 256;  // channels of queries and keys that are staged at once
 inline size_t softmax_attn_smem_bytes(int dim, int vdim) {
+  if (dim > kSmaxSlice) dim = kSmaxSlice;
   return sizeof(float) * (size_t(kSmaxRows) * dim + size_t(kSmaxKeys) * (dim + 1) + size_t(kSmaxKeys) * vdim + size_t(kSmaxRows) * kSmaxKeys +
                           3 * kSmaxRows);
 }
@@ -293,22 +343,26 @@ inline size_t softmax_attn_smem_bytes(int dim, int vdim) {
 template <typename T>
 __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(const SoftmaxAttnArgs<T> a) {
   extern __shared__ float smem[];
-  const int d = a.dim, dv = a.vdim, rep = a.heads / a.kv_heads;
-  float* sq = smem;                        // [16][d]
-  float* sk = sq + kSmaxRows * d;          // [32][d + 1]
-  float* sv = sk + kSmaxKeys * (d + 1);    // [32][dv]
+  const int d = a.dim, dv = a.vdim, rep = a.heads / a.kv_heads, maps = a.maps > 1 ? a.maps : 1, units = a.heads * maps;
+  const int ds = d < kSmaxSlice ? d : kSmaxSlice;  // channels staged at once
+  float* sq = smem;                        // [16][ds]
+  float* sk = sq + kSmaxRows * ds;         // [32][ds + 1]
+  float* sv = sk + kSmaxKeys * (ds + 1);   // [32][dv]
   float* sp = sv + kSmaxKeys * dv;         // [16][32]
   float* s_max = sp + kSmaxRows * kSmaxKeys;  // [16] running maximum
   float* s_sum = s_max + kSmaxRows;           // [16] running sum
   float* s_fix = s_sum + kSmaxRows;           // [16] factor that brings the old accumulators to the new maximum
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   griddep_wait();
-  const int r0 = a.tile_row0[blockIdx.x], nr = a.tile_row0[blockIdx.x + 1] - r0, h = blockIdx.y, g = h / rep;
+  const int r0 = a.tile_row0[blockIdx.x], nr = a.tile_row0[blockIdx.x + 1] - r0, u_all = blockIdx.y, h = u_all / maps, g = h / rep;
+  const int kh = a.wide ? 0 : g * maps + u_all % maps;  // key head
   const int p0 = a.pos[r0], grp = a.group[r0];  // row r0 + i has position p0 + i
   const int p_last = p0 + nr - 1;
-  int lo = 0;
-  if (a.window > 0 && p0 - a.window + 1 > 0) lo = p0 - a.window + 1;
-  for (int e = tid; e < nr * d; e += kSmaxThreads) sq[e] = act_f32(a.q[size_t(r0 + e / d) * a.heads * d + h * d + e % d]) * a.scale;
+  const int lo = smax_first(p0, a.window, a.chunk);
+  auto load_q = [&](int c0, int n) {
+    for (int e = tid; e < nr * n; e += kSmaxThreads) sq[(e / n) * ds + e % n] = act_f32(a.q[(size_t(r0 + e / n) * units + u_all) * d + c0 + e % n]) * a.scale;
+  };
+  if (ds == d) load_q(0, d);
   if (tid < kSmaxRows) {
     s_max[tid] = a.sink ? a.sink[h] : -INFINITY;
     s_sum[tid] = a.sink ? 1.0f : 0.0f;
@@ -325,30 +379,46 @@ __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(co
   const int begin = pooled ? 0 : lo, end = pooled ? nb_last - 1 : p_last, tpp = pooled ? a.pool_slots : a.tokens_per_page;
   const T* kpool = pooled ? a.kp_pages : a.k_pages;
   const T* vpool = pooled ? a.vp_pages : a.v_pages;
-  const size_t head_rows = size_t(g) * a.num_pages * tpp;
+  const size_t head_rows = size_t(g) * a.num_pages * tpp, key_rows = size_t(kh) * a.num_pages * tpp;
   for (int j0 = begin; j0 <= end; j0 += kSmaxKeys) {
     const int nk = end - j0 + 1 < kSmaxKeys ? end - j0 + 1 : kSmaxKeys;
     __syncthreads();
-    for (int e = tid; e < nk * d; e += kSmaxThreads) {
-      const int jj = e / d, c = e % d, j = j0 + jj;
-      const size_t row = head_rows + size_t(pages[j / tpp]) * tpp + j % tpp;
-      sk[jj * (d + 1) + c] = act_f32(kpool[row * d + c]);
-    }
     for (int e = tid; e < nk * dv; e += kSmaxThreads) {
       const int jj = e / dv, c = e % dv, j = j0 + jj;
       const size_t row = head_rows + size_t(pages[j / tpp]) * tpp + j % tpp;
       sv[jj * dv + c] = act_f32(vpool[row * dv + c]);
     }
-    __syncthreads();
-    for (int e = tid; e < nr * kSmaxKeys; e += kSmaxThreads) {
-      const int i = e / kSmaxKeys, jj = e % kSmaxKeys, j = j0 + jj, pi = p0 + i;
+    float sc[kSmaxRows * kSmaxKeys / kSmaxThreads];  // this thread's (row, key) pairs
+#pragma unroll
+    for (int w = 0; w < kSmaxRows * kSmaxKeys / kSmaxThreads; ++w) sc[w] = 0.0f;
+    for (int c0 = 0; c0 < d; c0 += ds) {
+      const int n = d - c0 < ds ? d - c0 : ds;
+      if (c0 > 0) __syncthreads();
+      if (ds < d) load_q(c0, n);
+      for (int e = tid; e < nk * n; e += kSmaxThreads) {
+        const int jj = e / n, c = e % n, j = j0 + jj;
+        const size_t row = key_rows + size_t(pages[j / tpp]) * tpp + j % tpp;
+        sk[jj * (ds + 1) + c] = act_f32(kpool[row * d + c0 + c]);
+      }
+      __syncthreads();
+#pragma unroll
+      for (int w = 0; w < kSmaxRows * kSmaxKeys / kSmaxThreads; ++w) {
+        const int e = tid + w * kSmaxThreads, i = e / kSmaxKeys, jj = e % kSmaxKeys;
+        if (i < nr && jj < nk) {
+          const float* qv = sq + i * ds;
+          const float* kv = sk + jj * (ds + 1);
+          for (int c = 0; c < n; ++c) sc[w] = fmaf(qv[c], kv[c], sc[w]);
+        }
+      }
+    }
+#pragma unroll
+    for (int w = 0; w < kSmaxRows * kSmaxKeys / kSmaxThreads; ++w) {
+      const int e = tid + w * kSmaxThreads, i = e / kSmaxKeys, jj = e % kSmaxKeys, j = j0 + jj, pi = p0 + i;
+      if (i >= nr) continue;
       float s = -INFINITY;
-      const bool seen = pooled ? j < smax_blocks_seen(pi, a.window, a.pool) : (j <= pi && (a.window <= 0 || pi - j < a.window));
+      const bool seen = pooled ? j < smax_blocks_seen(pi, a.window, a.pool) : (j <= pi && j >= smax_first(pi, a.window, a.chunk));
       if (jj < nk && seen) {
-        const float* qv = sq + i * d;
-        const float* kv = sk + jj * (d + 1);
-        s = 0.0f;
-        for (int c = 0; c < d; ++c) s = fmaf(qv[c], kv[c], s);
+        s = sc[w];
         if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
         if (!pooled) s -= slope * float(pi - j);
       }
@@ -391,6 +461,15 @@ __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(co
     const int o = tid + u * kSmaxThreads;
     if (o < nr * dv) {
       const int i = o / dv, c = o % dv;
+      if (maps > 1) {
+        const size_t at = size_t(r0 + i) * units + u_all;
+        a.part_o[at * dv + c] = acc[u];
+        if (c == 0) {
+          a.part_ml[at * 2] = s_max[i];
+          a.part_ml[at * 2 + 1] = s_sum[i];
+        }
+        continue;
+      }
       a.out[size_t(r0 + i) * a.ld_out + h * dv + c] = to_act<T>(acc[u] * a.out_scale / s_sum[i] * smax_gate(a.gate, a.ld_gate, r0 + i, h));
     }
   }
@@ -439,8 +518,7 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
   const int h = kvh * rep + (active ? unit / PARTS : 0), part = active ? unit % PARTS : 0;
   const int r0 = a.tile_row0[blockIdx.x], nr = a.tile_row0[blockIdx.x + 1] - r0;
   const int p0 = a.pos[r0], grp = a.group[r0], p_last = p0 + nr - 1;
-  int lo = 0;
-  if (a.window > 0 && p0 - a.window + 1 > 0) lo = p0 - a.window + 1;
+  const int lo = smax_first(p0, a.window, a.chunk);
   const int* pages = a.page_map + size_t(grp) * a.max_pages;
   const size_t head_rows = size_t(kvh) * a.num_pages * a.tokens_per_page;
   const int page_shift = (a.tokens_per_page & (a.tokens_per_page - 1)) == 0 ? __ffs(a.tokens_per_page) - 1 : -1;  // pages of 2^n tokens: no division per key
@@ -506,6 +584,7 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
   }
   const float slope = a.slopes ? a.slopes[h] : 0.0f;
   const int pi0 = p0 + g, pi1 = p0 + g + 8;
+  const int lo0 = smax_first(pi0, a.window, a.chunk), lo1 = smax_first(pi1, a.window, a.chunk), lo_last = smax_first(p_last, a.window, a.chunk);
   const int nb0 = smax_blocks_seen(pi0, a.window, a.pool), nb1 = smax_blocks_seen(pi1, a.window, a.pool);
   const int nb_first = smax_blocks_seen(p0, a.window, a.pool);
   const bool capped = a.softcap > 0.0f, sloped = a.slopes != nullptr;
@@ -527,7 +606,7 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
       const bool pooled = gt < pool_tiles;
       const int j0 = pooled ? gt * KT : lo + (gt - pool_tiles) * KT;
       // a tile whose every key every row of the query tile sees (most tiles of a long window) needs no masks
-      const bool every_key_seen = pooled ? j0 + KT <= nb_first : (j0 + KT - 1 <= p0 && (a.window <= 0 || p_last - j0 < a.window));
+      const bool every_key_seen = pooled ? j0 + KT <= nb_first : (j0 + KT - 1 <= p0 && j0 >= lo_last);
       float s[KT / 8][4];
 #pragma unroll
       for (int nb = 0; nb < KT / 8; ++nb) {
@@ -546,7 +625,7 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
           float sc = capped ? smax_softcap_scaled(s[nb][e], cap_mul, a.softcap) : s[nb][e] * a.scale;
           if (!every_key_seen || (sloped && !pooled)) {
             const int j = j0 + nb * 8 + 2 * t + (e & 1), pi = (e & 2) ? pi1 : pi0;
-            const bool seen = pooled ? j < ((e & 2) ? nb1 : nb0) : (j <= pi && (a.window <= 0 || pi - j < a.window));
+            const bool seen = pooled ? j < ((e & 2) ? nb1 : nb0) : (j <= pi && j >= ((e & 2) ? lo1 : lo0));
             if (sloped && !pooled) sc -= slope * float(pi - j);
             sc = seen ? sc : -INFINITY;
           }
@@ -670,8 +749,7 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
   const bool same_kv = a.k_pages == a.v_pages;  // the values are the cached keys' rows themselves: one copy of a tile serves both
   const int stage_elems = (same_kv ? 1 : 2) * KT * PITCH;
   const int pos = a.pos[row], grp = a.group[row];
-  int lo = 0;
-  if (a.window > 0 && pos - a.window + 1 > 0) lo = pos - a.window + 1;
+  const int lo = smax_first(pos, a.window, a.chunk);
   const int* pages = a.page_map + size_t(grp) * a.max_pages;
   const size_t head_rows = size_t(kvh) * a.num_pages * a.tokens_per_page;
   const int page_shift = (a.tokens_per_page & (a.tokens_per_page - 1)) == 0 ? __ffs(a.tokens_per_page) - 1 : -1;  // pages of 2^n tokens: no division per key
@@ -762,8 +840,8 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
       }
       // c[0], c[1]: key j0 + g, heads 2t, 2t + 1;  c[2], c[3]: key j0 + g + 8
       const int ja = j0 + g, jb = j0 + g + 8;
-      const bool sa_ = pooled ? ja < nb : (ja <= pos && (a.window <= 0 || pos - ja < a.window));
-      const bool sb_ = pooled ? jb < nb : (jb <= pos && (a.window <= 0 || pos - jb < a.window));
+      const bool sa_ = pooled ? ja < nb : ja <= pos;  // (no tile starts before the first visible key)
+      const bool sb_ = pooled ? jb < nb : jb <= pos;
 #pragma unroll
       for (int e = 0; e < 4; ++e) c[e] = a.softcap > 0.0f ? smax_softcap_scaled(c[e], cap_mul, a.softcap) : c[e] * a.scale;
       const float da = pooled ? 0.0f : float(pos - ja), db = pooled ? 0.0f : float(pos - jb);
@@ -880,6 +958,45 @@ __global__ void __launch_bounds__(128) softmax_attention_merge_kernel(const Soft
     }
     a.out[size_t(row) * a.ld_out + h * D + c] = __float2bfloat16_rn(acc * a.out_scale / L * gate);
   }
+}
+
+// maps == 2: o = a_0 - diff_lambda a_1 with a_m the merged result of unit 2 h + m; out[row, h] = diff_scale * unit(o); one warp per
+// (row, head)
+template <typename T>
+__global__ void __launch_bounds__(128) softmax_diff_merge_kernel(const SoftmaxAttnArgs<T> a) {
+  griddep_wait();
+  const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= a.rows * a.heads) return;
+  const int row = unit / a.heads, h = unit % a.heads, D = a.vdim, units = a.heads * 2;
+  float v[kSmaxMaxAcc * kSmaxThreads / kSmaxRows / 32];
+#pragma unroll
+  for (int i = 0; i < kSmaxMaxAcc * kSmaxThreads / kSmaxRows / 32; ++i) v[i] = 0.0f;
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    float M = -INFINITY, L = 0.0f;
+    for (int z = 0; z < a.splits; ++z) M = fmaxf(M, a.part_ml[((size_t(z) * a.rows + row) * units + 2 * h + m) * 2]);
+    for (int z = 0; z < a.splits; ++z) {
+      const float* ml = a.part_ml + ((size_t(z) * a.rows + row) * units + 2 * h + m) * 2;
+      if (ml[0] != -INFINITY) L += expf(ml[0] - M) * ml[1];
+    }
+    const float f = (m == 0 ? 1.0f : -a.diff_lambda) / L;
+    for (int z = 0; z < a.splits; ++z) {
+      const size_t base = (size_t(z) * a.rows + row) * units + 2 * h + m;
+      const float mz = a.part_ml[base * 2];
+      if (mz == -INFINITY) continue;
+      const float fz = f * expf(mz - M);
+#pragma unroll
+      for (int i = 0; i < kSmaxMaxAcc * kSmaxThreads / kSmaxRows / 32; ++i)
+        if (lane + i * 32 < D) v[i] = fmaf(fz, a.part_o[base * D + lane + i * 32], v[i]);
+    }
+  }
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kSmaxMaxAcc * kSmaxThreads / kSmaxRows / 32; ++i) ss = fmaf(v[i], v[i], ss);
+  const float inv = a.diff_scale / sqrtf(warp_sum(ss) / float(D) + a.eps);
+#pragma unroll
+  for (int i = 0; i < kSmaxMaxAcc * kSmaxThreads / kSmaxRows / 32; ++i)
+    if (lane + i * 32 < D) a.out[size_t(row) * a.ld_out + h * D + lane + i * 32] = to_act<T>(v[i] * inv);
 }
 
 }  // namespace mtx

@@ -36,7 +36,7 @@ QUERY_TILE_ROWS = 16  # rows of one query tile of the attention kernels (csrc/wi
 _LAYER_MATS = ("wqkv", "wo", "w_gate_up", "w_down", "w_in")
 _LAYER_VECS = ("bqkv", "q_norm", "k_norm", "dist_bias", "head_bias", "talk", "norm1", "norm1b", "norm2", "norm2b", "add_vector", "b_in", "bo",
                "conv1", "conv2")
-_ATTN_VECS = ("q_norm", "k_norm", "slopes", "sink")
+_ATTN_VECS = ("q_norm", "k_norm", "slopes", "sink", "temp", "talk")
 _LATENT_MATS = ("w_uq", "w_uk_t", "w_uv")
 _LATENT_VECS = ("q_norm", "kv_norm", "sink")
 _REC_VECS = ("decay_up_t", "decay_bias", "gate_bias", "out_norm", "conv_w", "a_log")
@@ -44,7 +44,7 @@ _REC_MATS = ("w_gate_up", "decay_up2")
 _SIDE_MATS = ("gate", "proj")
 _SIDE_VECS = ("norm",)
 _MOE_MATS = ("w_router", "w_gate_up", "w_down", "shared_gate_up", "shared_down")
-_MOE_VECS = ("correction",)
+_MOE_VECS = ("correction", "router_bias")
 
 
 def design_module(config):
@@ -65,6 +65,10 @@ def design_module(config):
     from . import ligidra
 
     return ligidra
+  if config.decoder_block == "fibelix":
+    from . import fibelix
+
+    return fibelix
   raise ValueError(f"decoder_block={config.decoder_block!r} is not a layered design")
 
 
@@ -223,9 +227,9 @@ class LayeredEngine(MaxEngine):
     ptr = lambda t: t.data_ptr() if t is not None else None
     slots = self.max_concurrent_decodes + 1  # (+ the parking slot of rows that belong to no live sequence)
 
-    def pools(G, d, dv):
-      kp = torch.zeros(G, pm.num_pages, pm.tokens_per_page, d, dtype=ct, device=dev)
-      vp = torch.zeros(G, pm.num_pages, pm.tokens_per_page, dv, dtype=ct, device=dev)
+    def pools(Gk, d, Gv, dv):
+      kp = torch.zeros(Gk, pm.num_pages, pm.tokens_per_page, d, dtype=ct, device=dev)
+      vp = torch.zeros(Gv, pm.num_pages, pm.tokens_per_page, dv, dtype=ct, device=dev)
       self._pools.append((kp, vp))
       return kp, vp
 
@@ -237,7 +241,7 @@ class LayeredEngine(MaxEngine):
       d.ff = int(l.get("ff", 0))
       states = ()
       if l["mixer"] == "window_sigmoid":
-        kp, vp = pools(l["kv_heads"], l["dim"], l["vdim"])
+        kp, vp = pools(l["kv_heads"], l["dim"], l["kv_heads"], l["vdim"])
         for k in ("heads", "kv_heads", "dim", "vdim", "window", "value_mix"):
           setattr(d, k, int(l[k]))
         for k in ("scale", "softcap", "value_lambda", "gain1", "gain2"):
@@ -259,9 +263,14 @@ class LayeredEngine(MaxEngine):
             kp, vp = self._pools[int(a["kv_from"])]
             self._pools.append(())
           else:
-            kp, vp = pools(a["kv_heads"], a["dim"], a["vdim"])
-          for k in ("heads", "kv_heads", "dim", "vdim", "window", "rot_dims", "values_are_keys", "rot_half", "shared_kv", "head_gate"):
+            # a key head of its own per map of a differential attention; heads whose scores are mixed read all key heads at once,
+            # so a token's keys lie side by side as one row
+            Gv, maps, dk = int(a["kv_heads"]), max(1, int(a.get("maps") or 1)), int(a["dim"])
+            Gk, dk = (1, Gv * dk) if a.get("talk") is not None else (Gv * maps, dk)
+            kp, vp = pools(Gk, dk, Gv, int(a["vdim"]))
+          for k in ("heads", "kv_heads", "dim", "vdim", "window", "rot_dims", "values_are_keys", "rot_half", "shared_kv", "head_gate", "chunk", "maps"):
             setattr(d.attn, k, int(a.get(k, 0)))
+          d.attn.diff_lambda, d.attn.diff_scale = float(a.get("diff_lambda", 0.0)), float(a.get("diff_scale", 0.0))
           d.attn.scale, d.attn.out_scale = float(a["scale"]), float(a["out_scale"])
           d.attn.rot_freq, d.attn.k_pages, d.attn.v_pages = ptr(a["rot_freq"]), kp.data_ptr(), vp.data_ptr()
           for k in _ATTN_VECS:
@@ -287,6 +296,7 @@ class LayeredEngine(MaxEngine):
           for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "rot_half"):
             setattr(d.latent, k, int(lat[k]))
           d.latent.scale, d.latent.pages = float(lat["scale"]), kp.data_ptr()
+          d.latent.window, d.latent.rot_amp = int(lat.get("window", 0)), float(lat.get("rot_amp", 1.0))
           for k in ("rot_freq",) + _LATENT_MATS + _LATENT_VECS:
             setattr(d.latent, k, ptr(lat.get(k)))
         else:
@@ -320,9 +330,9 @@ class LayeredEngine(MaxEngine):
           for k in ("experts", "top", "groups", "keep_groups", "ff", "shared_ff"):
             setattr(d.moe, k, int(m[k]))
           d.moe.limit, d.moe.shared_limit = float(m["limit"]), float(m["shared_limit"])
-          for k in ("w_router", "correction", "w_gate_up", "w_down", "shared_gate_up", "shared_down"):
+          for k in ("w_router", "correction", "router_bias", "w_gate_up", "w_down", "shared_gate_up", "shared_down"):
             setattr(d.moe, k, ptr(m.get(k)))
-          for k in ("score_softmax", "plain_weights", "act_silu"):
+          for k in ("score_softmax", "plain_weights", "act_silu", "chosen_softmax"):
             setattr(d.moe, k, int(m.get(k, 0)))
         sd = l.get("side")
         if sd:

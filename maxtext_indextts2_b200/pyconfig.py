@@ -36,8 +36,8 @@ _VALID_SAMPLING = ("greedy", "weighted", "nucleus", "topk")
 _VALID_AXIS_ORDER = ("0,1,2,3", "0,2,1,3")
 # Designs whose layers are listed one by one (`layer_specs`) and run on the layered engine (layered_engine.py), keyed by
 # decoder_block; ARCHITECTURES maps the "architecture" of a model folder's config.json to the block.
-LAYERED_BLOCKS = ("kifusun", "gugidra", "ginodra", "ligidra")
-ARCHITECTURES = {"Kifusun": "kifusun", "Gugidra": "gugidra", "Ginodra": "ginodra", "Ligidra": "ligidra"}
+LAYERED_BLOCKS = ("kifusun", "gugidra", "ginodra", "ligidra", "fibelix")
+ARCHITECTURES = {"Kifusun": "kifusun", "Gugidra": "gugidra", "Ginodra": "ginodra", "Ligidra": "ligidra", "Fibelix": "fibelix"}
 
 
 def _string_to_bool(s: str) -> bool:
@@ -142,6 +142,10 @@ def _validate_layered(keys: dict) -> None:
     ligidra.validate_layer_specs(keys["layer_specs"])
     if int(keys["token_side_dim"]) < 0:
       raise ValueError("token_side_dim must not be negative")
+  if keys["decoder_block"] == "fibelix":
+    from . import fibelix
+
+    fibelix.validate_layer_specs(keys["layer_specs"])
 
 
 def _validate(keys: dict) -> None:
@@ -314,6 +318,10 @@ def from_model_dict(model: dict, **overrides) -> HyperParameters:
     from . import ligidra
 
     keys = ligidra.config_keys(model)
+  elif block == "fibelix":
+    from . import fibelix
+
+    keys = fibelix.config_keys(model)
   keys.update(decoder_block=block, attention="paged", scan_layers=False, weight_dtype="bfloat16")
   keys.update(overrides)
   if "max_prefill_predict_length" not in overrides:  # any prompt that fits the sequence
