@@ -66,7 +66,7 @@ def parse_args():
   ap.add_argument("--no-verify", action="store_true", help="skip the oracle check of one step of the timed state")
   ap.add_argument("--prompt-len", type=int, default=4000, help="--mode prefill: prompt tokens (BASELINE configs[3]: 4000 of P = 4096)")
   ap.add_argument("--size", default="all", help="--mode layered: one of the sizes of LAYERED_SIZES, or all")
-  ap.add_argument("--design", default="kifusun", choices=["kifusun", "gugidra", "ginodra", "ligidra"], help="--mode layered: the layered design that is measured beside gemma3")
+  ap.add_argument("--design", default="kifusun", choices=["kifusun", "gugidra", "ginodra", "ligidra", "fibelix"], help="--mode layered: the layered design that is measured beside gemma3")
   ap.add_argument("--mode", default="batch", choices=["batch", "vocab-parallel", "prefill", "layered"],
                   help="batch: request-batch partitioned, no collective (default); vocab-parallel: every GPU decodes the same --batch slots, "
                        "the logits projection is sharded over the GPUs and one NCCL all-gather carries the per-shard candidates")
@@ -614,7 +614,7 @@ def run_layered(args):
   """--mode layered: prefill and decode throughput of a layered design (--design) on the layered engine beside the gemma3 block
   (the closest existing model: softmax attention with rotary positions and grouped key heads, norms before and after every
   sublayer, gated feed-forward) at equal layer sizes, both through MaxEngine.  One JSON line per size."""
-  from maxtext_indextts2_b200 import ginodra, gugidra, kifusun, ligidra, maxengine, pyconfig
+  from maxtext_indextts2_b200 import fibelix, ginodra, gugidra, kifusun, ligidra, maxengine, pyconfig
 
   D = args.design  # (the keys of the output line carry the design's name)
   names = list(LAYERED_SIZES) if args.size == "all" else [args.size]
@@ -624,6 +624,7 @@ def run_layered(args):
     P, B, C, L = z["prompt"], z["batch"], z["context"], z["layers"]
     T = max(P, C) + 64
     tpp = 64
+    ctx = C  # tokens that every slot of the layered design holds in the decode measurement
     out = {"metric": "layered model: prefill tokens/s and decode tokens/s beside gemma3 at equal size", "mode": "layered", "size": name, "geometry": z,
            "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic, random weights", "l2": "flushed between timed iterations"}
     # ---- the layered design ----
@@ -656,6 +657,23 @@ def run_layered(args):
                 ligidra.attention_layer(H, G, d, window=W, pool=16, softcap=50.0, rot_scaling=scaling, kv_from=0, mlp=ff()),
                 ligidra.delta_layer(H, G, d // 2, d, taps=4, per_channel=True, rank=64, mlp=ff())][:L]
       model = ligidra.model_dict(z["width"], z["vocab"], layers, side_dim=z["width"] // 8)
+    elif D == "fibelix":
+      # Fibelix at the same sizes, one layer of each kind: a differential attention (gemma3's heads, each split into two maps of half
+      # the size, over values of the full size), a latent attention (cached rows as wide as two of gemma3's key heads, gemma3's window), a
+      # talking attention with gemma3's heads, a differential attention that reads the first one's cache; every layer with a routed
+      # feed-forward of gemma3's active size (16 experts of ff / 4, four per token).  Chunks are twice gemma3's window, so that a prompt's
+      # tokens see as many keys on average, and the decode slots stand in the middle of a chunk
+      H, G, d, F, W = z["heads"], z["kv_heads"], z["dim"], z["ff"], z["window"]
+      row = min(256, 2 * d)
+      ff = lambda: fibelix.moe_ff(16, 4, F // 4)
+      yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+      layers = [fibelix.differential_layer(H, G, d // 2, d, chunk=2 * W, mlp=ff()),
+                fibelix.latent_layer(H, d // 2, row // 4, d // 2, z["width"] // 2, row - row // 4, window=W, rot_scaling=yarn, mlp=ff()),
+                fibelix.talking_layer(H, G, d, chunk=2 * W, rot_factor=8.0, mlp=ff()),
+                fibelix.differential_layer(H, G, d // 2, d, chunk=2 * W, kv_from=0, mlp=ff())][:L]
+      model = fibelix.model_dict(z["width"], z["vocab"], layers)
+      ctx = (C // (2 * W) * 2 + 1) * W
+      T = max(T, ctx + 64)
     else:
       # Gugidra at the same sizes: attention + mLSTM layers and GLA layers in turn; the attention has gemma3's heads (no window: the
       # design has none), the recurrences half as many key channels per head; dense feed-forwards of gemma3's size in turn with
@@ -665,7 +683,7 @@ def run_layered(args):
       layers = [gugidra.parallel_layer(H, G, d, H // 2, d // 2, d, mlp=ffs[(i // 2) % 2]) if i % 2 == 0 else gugidra.gla_layer(H, d // 2, d, mlp=ffs[((i + 1) // 2) % 2])
                 for i in range(L)]
       model = gugidra.model_dict(z["width"], z["vocab"], layers)
-    pages = B * ((C + 8 + tpp - 1) // tpp) + (P + tpp - 1) // tpp + 2
+    pages = B * ((ctx + 16 + tpp - 1) // tpp) + (P + tpp - 1) // tpp + 2
     cfg = pyconfig.from_model_dict(model, dtype="bfloat16", per_device_batch_size=B, max_target_length=T, pagedattn_tokens_per_page=tpp,
                                    pagedattn_num_pages=pages, max_step_rows=max(P, B))
     engine = maxengine.MaxEngine(cfg)
@@ -682,7 +700,8 @@ def run_layered(args):
     out[D + "_prefill_ms"], out[D + "_prefill_tokens_per_s"] = ms, P / ms * 1e3
     out[D + "_prefill_launches"] = int(engine.lib.mtx_launch_count() - n0) // (steps + warmup)
     engine.release_pages(0)
-    state = engine.fill_synthetic_context([C] * B)  # every slot holds a C-token context (only the cache and state traffic matters)
+    state = engine.fill_synthetic_context([ctx] * B)  # every slot holds a context of that many tokens (only the cache and state traffic matters)
+    out[D + "_decode_context"] = ctx
 
     def k_decode():
       engine.generate(params, state)

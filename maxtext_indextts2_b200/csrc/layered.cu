@@ -715,25 +715,27 @@ int launch_multi_prefill_t(const SoftmaxAttnArgs<bf16>& sa, const MultiMmaPlan& 
     MTX_CUDA(cudaFuncSetAttribute(multi_attention_prefill_kernel<DV16, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(p.smem)));
     have = p.smem;
   }
-  return launch(multi_attention_prefill_kernel<DV16, KT>, dim3((n_tiles + p.rt - 1) / p.rt, sa.kv_heads * p.chunks), dim3(kMatThreads), p.smem, st, sa, n_tiles, p.uw,
+  return launch(multi_attention_prefill_kernel<DV16, KT>, dim3((n_tiles + p.rt - 1) / p.rt, sa.kv_heads * p.chunks), dim3(p.warps * 32), p.smem, st, sa, n_tiles, p.uw,
                 p.rt, p.chunks);
 }
 
 int launch_multi_prefill(const SoftmaxAttnArgs<bf16>& sa, const MultiMmaPlan& p, int n_tiles, cudaStream_t st) {
   if (p.dv16 == 4 && p.kt == 64) return launch_multi_prefill_t<4, 64>(sa, p, n_tiles, st);
-  if (p.dv16 == 4) return launch_multi_prefill_t<4, 32>(sa, p, n_tiles, st);
+  if (p.dv16 == 4 && p.kt == 32) return launch_multi_prefill_t<4, 32>(sa, p, n_tiles, st);
+  if (p.kt == 16 && p.dv16 <= 8) return launch_multi_prefill_t<8, 16>(sa, p, n_tiles, st);
+  if (p.kt == 16) return launch_multi_prefill_t<16, 16>(sa, p, n_tiles, st);
   if (p.dv16 == 8) return launch_multi_prefill_t<8, 32>(sa, p, n_tiles, st);
   return launch_multi_prefill_t<16, 32>(sa, p, n_tiles, st);
 }
 
-template <int SPW, int DV16>
+template <int NV, int DV16>
 int launch_multi_decode_t(const SoftmaxAttnArgs<bf16>& sa, const MultiDecodePlan& p, cudaStream_t st) {
   static size_t have = 0;  // per instantiation
   if (p.smem > 48 * 1024 && p.smem > have) {
-    MTX_CUDA(cudaFuncSetAttribute(multi_attention_decode_kernel<SPW, DV16>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(p.smem)));
+    MTX_CUDA(cudaFuncSetAttribute(multi_attention_decode_kernel<NV, DV16>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(p.smem)));
     have = p.smem;
   }
-  return launch(multi_attention_decode_kernel<SPW, DV16>, dim3(sa.rows, p.groups * p.chunks, sa.splits), dim3(128), p.smem, st, sa, p.sets, p.sg, p.chunks);
+  return launch(multi_attention_decode_kernel<NV, DV16>, dim3(sa.rows, p.groups * p.chunks, sa.splits), dim3(128), p.smem, st, sa, p.sg, p.chunks);
 }
 
 // key splits as for the other single-token kernel: waves of resident CTAs x (key tiles per split + a split's start-up of two tiles)
@@ -757,12 +759,12 @@ int launch_multi_decode(mtx_layered* e, SoftmaxAttnArgs<bf16>& sa, const MultiDe
   }
   if (force >= 1 && force <= 4 && size_t(force) * sa.rows <= e->attn_part_rows) sa.splits = force;
   int rc = MTX_ERR_UNSUPPORTED;
-  if (p.spw == 1 && p.dv16 == 4) rc = launch_multi_decode_t<1, 4>(sa, p, st);
-  else if (p.spw == 1 && p.dv16 == 8) rc = launch_multi_decode_t<1, 8>(sa, p, st);
-  else if (p.spw == 1) rc = launch_multi_decode_t<1, 16>(sa, p, st);
-  else if (p.dv16 == 4) rc = launch_multi_decode_t<2, 4>(sa, p, st);
-  else if (p.dv16 == 8) rc = launch_multi_decode_t<2, 8>(sa, p, st);
-  else rc = launch_multi_decode_t<2, 16>(sa, p, st);
+  if (p.nv == 1 && p.dv16 == 4) rc = launch_multi_decode_t<1, 4>(sa, p, st);
+  else if (p.nv == 1 && p.dv16 == 8) rc = launch_multi_decode_t<1, 8>(sa, p, st);
+  else if (p.nv == 1) rc = launch_multi_decode_t<1, 16>(sa, p, st);
+  else if (p.nv == 2 && p.dv16 == 4) rc = launch_multi_decode_t<2, 4>(sa, p, st);
+  else if (p.nv == 2) rc = launch_multi_decode_t<2, 8>(sa, p, st);
+  else rc = launch_multi_decode_t<4, 4>(sa, p, st);
   MTX_TRY(rc);
   if (sa.maps > 1) return launch(softmax_diff_merge_kernel<bf16>, dim3((sa.rows * sa.heads + 3) / 4), dim3(128), 0, st, sa);
   if (sa.splits > 1) return launch(softmax_attention_merge_kernel, dim3((sa.rows * sa.heads + 3) / 4), dim3(128), 0, st, sa);
@@ -788,7 +790,7 @@ int run_softmax_attention(mtx_layered* e, SoftmaxAttnArgs<T>& sa, const mtx_ragg
         if (b.n_tiles == sa.rows && decode_arm) return launch_softmax_decode(e, sa, plan.d16, st);
         return launch_softmax_mma(e, sa, plan, b.n_tiles, b.n_tiles == sa.rows, st);
       }
-      if (sa.pool == 0 && !sa.slopes && sa.softcap == 0.0f) {
+      if (sa.pool == 0 && !sa.slopes && sa.softcap == 0.0f && sa.scale > 0.0f) {
         const bool same_kv = sa.k_pages == sa.v_pages;
         if (b.n_tiles == sa.rows) {
           const MultiDecodePlan p = multi_decode_plan(sa.heads, sa.kv_heads, sa.dim, sa.vdim, maps, sa.wide != 0, same_kv);

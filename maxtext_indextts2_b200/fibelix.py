@@ -291,5 +291,5 @@ def latent_layer(heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_
   m: Dict[str, Any] = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank,
                        "rot": {"base": rot_base, "dims": rot_dim}, "scale": scale or (dim + rot_dim) ** -0.5}
   if rot_scaling:
-    m["rot"]["scaling"] = rot_scaling
+    m["rot"]["scaling"] = dict(rot_scaling)
   return _mixer("latent_attention", m, window, mlp)
