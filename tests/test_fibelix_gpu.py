@@ -385,6 +385,8 @@ SIZES = {
     "many_heads_on_one_key_head": lambda: model([tlk(heads=10, kv_heads=1, dim=8, vdim=8), dif(heads=9, kv_heads=1, dim=8, vdim=8), lat(heads=10)]),
     "three_and_five_key_heads": lambda: model([tlk(heads=6, kv_heads=3, dim=16, vdim=24), dif(heads=6, kv_heads=3, dim=8, vdim=24), tlk(heads=5, kv_heads=5, dim=8, vdim=16),
                                                dif(heads=10, kv_heads=5, dim=16, vdim=8)]),
+    "three_query_heads_per_key_head": lambda: model([tlk(heads=9, kv_heads=3, dim=16, vdim=16), dif(heads=9, kv_heads=3, dim=8, vdim=16), dif(heads=15, kv_heads=3, dim=8, vdim=16)]),
+    "one_expert": lambda: model([lat(moe(1, 1, 12)), tlk(moe(2, 2, 8))]),
     "value_size_over_key_size": lambda: model([tlk(dim=8, vdim=40), dif(dim=8, vdim=72)]),
     "key_size_over_value_size": lambda: model([tlk(dim=40, vdim=8, rot_dims=40), dif(dim=40, vdim=8)]),
     "rotation_of_two_channels": lambda: model([tlk(rot_dims=2), lat(rot_dim=2)]),
@@ -438,13 +440,13 @@ SHAPES = {
     "talking_8x128_on_8_values_128": lambda: tlk(heads=8, kv_heads=8, dim=128, vdim=128, chunk=80, rot_dims=64),
     "differential_4x32_on_2": lambda: dif(heads=4, kv_heads=2, dim=32, vdim=64, chunk=70),
     "differential_16x16_on_1": lambda: dif(heads=16, kv_heads=1, dim=16, vdim=32, chunk=128),
-    "differential_3x48_on_3": lambda: dif(heads=3, kv_heads=3, dim=48, vdim=96, chunk=100),
+    "differential_3x56_on_3_values_112": lambda: dif(heads=3, kv_heads=3, dim=56, vdim=112, chunk=100),
     "differential_12x40_on_4_values_56": lambda: dif(heads=12, kv_heads=4, dim=40, vdim=56, chunk=37),
     "differential_10x8_on_2_values_24": lambda: dif(heads=10, kv_heads=2, dim=8, vdim=24, chunk=64),
     "differential_2x128_on_1_values_256": lambda: dif(heads=2, kv_heads=1, dim=128, vdim=256, chunk=90),
     "latent_rows_of_40": lambda: lat(heads=4, dim=16, rot_dim=8, vdim=16, q_rank=24, kv_rank=32, window=50),
     "latent_rows_of_104": lambda: lat(heads=9, dim=24, rot_dim=24, vdim=32, q_rank=24, kv_rank=80, window=70),
-    "latent_rows_of_128": lambda: lat(heads=6, dim=32, rot_dim=32, vdim=32, q_rank=48, kv_rank=96, window=33),
+    "latent_rows_of_128": lambda: lat(heads=5, dim=24, rot_dim=16, vdim=24, q_rank=48, kv_rank=112, window=33),
     "latent_rows_of_192": lambda: lat(heads=3, dim=32, rot_dim=64, vdim=32, q_rank=48, kv_rank=128, window=0),
 }
 
