@@ -5,7 +5,7 @@
 // A UNIT is one softmax: a (query head, map) pair.  The units of one value head ("its units") share that head's value rows; their
 // key rows are, per map, one slice of `dim` channels (wide: all units read the same rows).
 //
-//   multi_attention_prefill_kernel<DV16, KT>   rows in portions.  CTA of eight warps = `rt` query tiles (16 rows each, consecutive
+//   multi_attention_prefill_kernel<DV16, KT>   rows in portions.  CTA of eight warps (four with 16-key tiles, for the widest keys) = `rt` query tiles (16 rows each, consecutive
 //                        entries of the host's table) x `uw` units of a value head: a warp owns one (tile, unit) pair, S = Q K^T and
 //                        O += P V on mma.sync m16n8k16 with fp32 accumulators, running maximum and sum in fp32 registers.  Tiles
 //                        that continue one another share the staged keys and values (cp.async double buffer through the page map);
