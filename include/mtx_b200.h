@@ -380,11 +380,17 @@ int mtx_engine_rebind_state(mtx_engine* e, const mtx_decode_state* s);
                                The embedding output is normed with mtx_layered_config.embed_norm (if any), the final norm uses its
                                weight as stored.  One mixer per layer: attn, latent or rec (MTX_REC_GDELTA); conv1 may be NULL (the mixer
                                then reads h itself); b_in and bo are added where the projections are */
+#define MTX_NORM_OUT_LAYER 4 /* layer norms on the sublayers' outputs, which read x itself:  x += ln(mixer(x)) * norm1 + norm1b;
+                               x += ln(ff(x)) * norm2 + norm2b if the layer has a feed-forward, ln(y) = (y - mean(y)) / sqrt(mean((y -
+                               mean(y))^2) + eps).  (A layer scale s is folded into the vectors: norm1 = s w, norm1b = s b.)  The
+                               mixer is MTX_MIXER_COMPOSITE: attn and / or rec (MTX_REC_DECAY).  The final norm is a layer norm
+                               with mtx_layered_config.final_norm and final_norm_b */
 
 #define MTX_FF_GELU_GATED 0    /* down(gelu_tanh(gate x) * up x) */
 #define MTX_FF_CLAMPED_GATED 1 /* down(g s(1.702 g) (u + 1)), g = min(gate x, limit), u = clamp(up x, -limit, limit), s = sigmoid */
 #define MTX_FF_MOE 2           /* routed experts of the clamped form plus an optional shared one (mtx_moe_desc) */
 #define MTX_FF_RELU2 3         /* down(relu(up x)^2); MTX_NORM_PARALLEL layers: w_gate_up = up [ff, width], down is part of wo */
+#define MTX_FF_GELU 4          /* down(gelu_tanh(up x)); w_gate_up = up [ff, width] */
 
 /* Causal softmax attention over the paged cache (csrc/softmax_attention.cuh).  Its projection rows in the layer's w_in are
  * [q: heads*dim | k: kv_heads*dim | v: kv_heads*vdim unless values_are_keys]. */
@@ -434,6 +440,11 @@ typedef struct {
   const float* temp;       /* [heads] or NULL: head h's score is multiplied by temp[h] (before the mixing) */
   const float* talk;       /* [heads, heads] or NULL: before the softmax score_h becomes sum_g talk[h, g] * score_g.  The key pool is
                               then [1, num_pages, tokens_per_page, kv_heads*dim]: a token's keys of all key heads side by side */
+  /* -- MTX_NORM_OUT_LAYER layers, neither together with pooled blocks, slopes, chunks, two maps or mixed scores -- */
+  int32_t keep_first;      /* F > 0 (needs a window): beside the window's tokens every query sees the first F tokens of its sequence, at
+                              their true positions */
+  int32_t value_gate;      /* 1: heads*vdim more projection rows follow the attention's own: the concatenated heads are multiplied,
+                              channel by channel, by sigmoid(row) */
 } mtx_softmax_attn_desc;
 
 /* Attention through latents (csrc/latent_attention.cuh): queries q = w_uq rmsnorm(dq x) laid out per head as [dim plain | rot_dim
@@ -476,6 +487,8 @@ typedef struct {
                            parts of the matmul dtype so that the product keeps fp32 accuracy).  Output gate: gate_rank == 0: heads*vdim
                            projection rows; else w_gate_up (gate_rank rows of the projection).  Projection rows: [q: kv_heads*dim |
                            k: kv_heads*dim | v: heads*vdim | beta: heads | decay: heads or decay_rank | gate: heads*vdim or gate_rank] */
+#define MTX_REC_DECAY 5 /* decayed sums with one constant per head (lightning attention): S <- head_decay[h] S + k v^T, o = S^T q; q, k and v
+                           pass silu.  Projection rows: [q | k | v | output gate: heads*vdim] */
 
 /* A linear recurrence with a matrix state per head (csrc/recurrent_mixers.cuh).  State, decays and gates are fp32.  Its
  * projection rows in w_in follow the attention's: [q: heads*dim | k: heads*dim | v: heads*vdim | output gate: heads*vdim |
@@ -507,6 +520,9 @@ typedef struct {
   float* conv_state;       /* [state slots, conv_taps - 1, 2*kv_heads*dim + heads*vdim]: the projection row of position p at p % (conv_taps - 1) */
   const float* a_log;      /* [heads] */
   const void* w_gate_up;   /* [heads*vdim, gate_rank] in the matmul dtype, or NULL */
+  /* -- MTX_REC_DECAY -- */
+  const float* head_decay; /* [heads] */
+  int32_t norm_whole;      /* 1: o is divided by the root mean square over all heads together instead of head by head */
 } mtx_recurrent_desc;
 
 /* Routed feed-forward (csrc/moe.cuh): scores s = sigmoid(router x) (score_softmax: softmax over all experts); an expert is chosen by s + correction among the experts of
@@ -530,6 +546,12 @@ typedef struct {
   int32_t chosen_softmax;  /* 1: experts are chosen by their logits (+ correction), and the weights are the softmax over the chosen
                               experts' logits alone (score_softmax / plain_weights are then not read) */
   const float* router_bias; /* [experts] or NULL: added to the router's logits */
+  /* -- MTX_NORM_OUT_LAYER layers -- */
+  int32_t groups_max;      /* 1: a group's score is its largest choice score (not the sum of its two largest) */
+  int32_t identity;        /* router outputs beyond `experts` whose expert's output is the feed-forward's input itself: w_router and
+                              correction have experts + identity entries, and the groups are formed over all of them */
+  int32_t shared_gate;     /* 1: the shared expert's output is multiplied by sigmoid(<row, x>), one number per token; the row is the one
+                              after the router's outputs in w_router */
 } mtx_moe_desc;
 
 typedef struct {
@@ -558,7 +580,7 @@ typedef struct {
   void* k_pages;        /* [G, num_pages, tokens_per_page, dim] */
   void* v_pages;        /* [G, num_pages, tokens_per_page, vdim] */
   /* -- the fields above describe MTX_MIXER_WINDOW_SIGMOID layers with MTX_NORM_OUT_GAIN; the ones below every other kind -- */
-  int32_t norm_style;   /* MTX_NORM_* */
+  int32_t norm_style;   /* MTX_NORM_* (MTX_NORM_OUT_LAYER: norm1 / norm1b and norm2 / norm2b are the weights and biases) */
   int32_t ff_kind;      /* MTX_FF_* */
   int32_t n_in;         /* MTX_MIXER_COMPOSITE: rows of w_in (the sub-mixers' rows, then zero rows up to a tile edge if any) */
   int32_t add_embedding; /* 1: before this layer x += the embedding output of the same row */
@@ -616,6 +638,8 @@ typedef struct {
   const float* embed_norm;     /* [width] or NULL: the embedding output becomes unit(.) * embed_norm */
   const void* side_embed;      /* [vocab, side_width] rows of the per-layer token inputs, or NULL */
   int32_t side_width;
+  /* -- MTX_NORM_OUT_LAYER models -- */
+  const float* final_norm_b;   /* [width] */
 } mtx_layered_config;
 
 typedef struct {

@@ -109,9 +109,9 @@ class DecodeState(ctypes.Structure):
 
 
 MIXER_WINDOW_SIGMOID, MIXER_COMPOSITE = 1, 2
-NORM_OUT_GAIN, NORM_SANDWICH, NORM_PARALLEL, NORM_PRE = 0, 1, 2, 3
-FF_GELU_GATED, FF_CLAMPED_GATED, FF_MOE, FF_RELU2 = 0, 1, 2, 3
-REC_GLA, REC_MLSTM, REC_DELTA, REC_GDELTA = 1, 2, 3, 4
+NORM_OUT_GAIN, NORM_SANDWICH, NORM_PARALLEL, NORM_PRE, NORM_OUT_LAYER = 0, 1, 2, 3, 4
+FF_GELU_GATED, FF_CLAMPED_GATED, FF_MOE, FF_RELU2, FF_GELU = 0, 1, 2, 3, 4
+REC_GLA, REC_MLSTM, REC_DELTA, REC_GDELTA, REC_DECAY = 1, 2, 3, 4, 5
 
 
 class SoftmaxAttnDesc(ctypes.Structure):
@@ -129,6 +129,7 @@ class SoftmaxAttnDesc(ctypes.Structure):
       + [(n, ctypes.c_int32) for n in ("chunk", "maps")]
       + [(n, ctypes.c_float) for n in ("diff_lambda", "diff_scale")]
       + [(n, ctypes.c_void_p) for n in ("temp", "talk")]
+      + [(n, ctypes.c_int32) for n in ("keep_first", "value_gate")]
   )
 
 
@@ -152,7 +153,8 @@ class RecurrentDesc(ctypes.Structure):
       + [(n, ctypes.c_void_p) for n in ("decay_up_t", "decay_bias", "gate_bias", "out_norm", "state_s", "state_n", "state_m")]
       + [(n, ctypes.c_float) for n in ("decay_rate", "key_eps")]
       + [(n, ctypes.c_int32) for n in ("kv_heads", "conv_taps", "gate_rank")]
-      + [(n, ctypes.c_void_p) for n in ("conv_w", "conv_state", "a_log", "w_gate_up")]
+      + [(n, ctypes.c_void_p) for n in ("conv_w", "conv_state", "a_log", "w_gate_up", "head_decay")]
+      + [("norm_whole", ctypes.c_int32)]
   )
 
 
@@ -165,6 +167,7 @@ class MoeDesc(ctypes.Structure):
       + [(n, ctypes.c_void_p) for n in ("w_router", "correction", "w_gate_up", "w_down", "shared_gate_up", "shared_down")]
       + [(n, ctypes.c_int32) for n in ("score_softmax", "plain_weights", "act_silu", "chosen_softmax")]
       + [("router_bias", ctypes.c_void_p)]
+      + [(n, ctypes.c_int32) for n in ("groups_max", "identity", "shared_gate")]
   )
 
 
@@ -197,7 +200,7 @@ class LayeredConfig(ctypes.Structure):
       + [(n, ctypes.c_float) for n in ("eps", "embed_scale", "final_gain")]
       + [(n, ctypes.c_void_p) for n in ("embedding", "head", "final_norm")]
       + [("logit_softcap", ctypes.c_float), ("norm_groups", ctypes.c_int32), ("logit_scale", ctypes.c_float)]
-      + [("embed_norm", ctypes.c_void_p), ("side_embed", ctypes.c_void_p), ("side_width", ctypes.c_int32)]
+      + [("embed_norm", ctypes.c_void_p), ("side_embed", ctypes.c_void_p), ("side_width", ctypes.c_int32), ("final_norm_b", ctypes.c_void_p)]
   )
 
 

@@ -17,6 +17,9 @@
 //   pre_norm_step_kernel    pre-norm layers: x = unit(x) * w0 (optional); x += y or x += unit(y) * wy (optional); a copy of x in the matmul
 //                           dtype (optional); unit(x) * w to the fp32 plane of normed rows and / or the matmul dtype (optional), or,
 //                           in steps of single tokens, straight through the next mixer's input convolution and into its ring
+//   out_layer_norm_kernel   x += ln(y) * w + b (a layer norm on the sublayer's OUTPUT) and its copy in the matmul dtype; y is a plane (fp32, or
+//                           bf16 as a tcgen05 GEMM left it) or the weighted sum of a routed feed-forward's experts, added up on the way
+//   layer_norm_rows_kernel  ln(x) * w + b of a gathered subset of rows
 //   side_act_kernel         act = gelu_tanh(gate) * table[token, col ..]: the gated rows of a per-layer token input
 //
 // Everything here is fp32 arithmetic; T is the dtype the matrix products and the cache use (bf16, or float for a float32 engine).
@@ -411,6 +414,132 @@ __global__ void __launch_bounds__(256) pre_norm_step_kernel(const PreNormArgs a,
       if (ring > 0) cv.state[(size_t(grp) * ring + p % ring) * W + c] = hv;  // (the slot of position p - ring, read just above by this thread)
     }
   }
+}
+
+struct OutLayerNormArgs {
+  const float* y;        // [rows, width] the sublayer's output, or null:
+  const bf16* y_bf16;    // ... as bf16, or null (both null: nothing but the experts below)
+  const float* shared_gate;  // [rows, ld_gate]: y is multiplied by sigmoid(shared_gate[row]), or null
+  int ld_gate;
+  // a routed feed-forward (top > 0): + sum over the row's choices, in their order, of weight * (chosen < experts: row slot_of of expert_y,
+  // else the row of x itself)
+  const float* expert_y;
+  const int* slot_of;
+  const int* chosen;
+  const float* weight;
+  int top, experts;
+  const float* w;        // [width]
+  const float* b;        // [width]
+  float* x;              // [rows, width]
+  float eps;
+  int width;
+};
+
+constexpr int kOutLnVec = 32;  // registers of a thread for its part of the row: width <= 256 * kOutLnVec
+
+// one CTA per row; the row stays in registers between the reductions (mean, then the squared deviations).  V = 4: the row moves in
+// groups of four channels (width a multiple of 4), V = 1: any width
+template <typename T, int V>
+__global__ void __launch_bounds__(256) out_layer_norm_kernel(const OutLayerNormArgs a, T* xa) {
+  __shared__ float red[8];
+  constexpr int N = kOutLnVec / V;
+  griddep_wait();
+  const int r = blockIdx.x, W = a.width;
+  float* xr = a.x + size_t(r) * W;
+  auto load = [&](const float* p, int c, float (&v)[V]) {
+    if constexpr (V == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(p + c);
+      v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
+    } else {
+      v[0] = p[c];
+    }
+  };
+  const float sg = a.shared_gate ? 1.0f / (1.0f + expf(-a.shared_gate[size_t(r) * a.ld_gate])) : 1.0f;
+  float yv[N][V];
+  float sum = 0.0f;
+#pragma unroll
+  for (int u = 0; u < N; ++u) {
+    const int c = (threadIdx.x + u * 256) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) yv[u][e] = 0.0f;
+    if (c < W) {
+      if (a.y) {
+        load(a.y + size_t(r) * W, c, yv[u]);
+      } else if (a.y_bf16) {
+        const bf16* yb = a.y_bf16 + size_t(r) * W + c;
+        if constexpr (V == 4) {
+          const uint2 q = *reinterpret_cast<const uint2*>(yb);
+          const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+          yv[u][0] = lo.x, yv[u][1] = lo.y, yv[u][2] = hi.x, yv[u][3] = hi.y;
+        } else {
+          yv[u][0] = __bfloat162float(yb[0]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) yv[u][e] *= sg;
+      for (int k = 0; k < a.top; ++k) {
+        const size_t at = size_t(r) * a.top + k;
+        float v[V];
+        load(a.chosen[at] < a.experts ? a.expert_y + size_t(a.slot_of[at]) * W : xr, c, v);
+        const float wt = a.weight[at];
+#pragma unroll
+        for (int e = 0; e < V; ++e) yv[u][e] = fmaf(wt, v[e], yv[u][e]);
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) sum += yv[u][e];
+    }
+  }
+  const float mean = block_sum(sum, red) / float(W);
+  float ss = 0.0f;
+#pragma unroll
+  for (int u = 0; u < N; ++u)
+    if ((threadIdx.x + u * 256) * V < W) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        yv[u][e] -= mean;
+        ss = fmaf(yv[u][e], yv[u][e], ss);
+      }
+    }
+  const float f = 1.0f / sqrtf(block_sum(ss, red) / float(W) + a.eps);
+#pragma unroll
+  for (int u = 0; u < N; ++u) {
+    const int c = (threadIdx.x + u * 256) * V;
+    if (c < W) {
+      float v[V], w[V], b[V];
+      load(xr, c, v);
+      load(a.w, c, w);
+      load(a.b, c, b);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += fmaf(yv[u][e] * f, w[e], b[e]);
+      if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(xr + c) = make_float4(v[0], v[1], v[2], v[3]);
+        if constexpr (sizeof(T) == 2) {
+          const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+          *reinterpret_cast<uint2*>(xa + size_t(r) * W + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+          *reinterpret_cast<float4*>(xa + size_t(r) * W + c) = make_float4(v[0], v[1], v[2], v[3]);
+        }
+      } else {
+        xr[c] = v[0];
+        xa[size_t(r) * W + c] = to_act<T>(v[0]);
+      }
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) layer_norm_rows_kernel(const float* x, const int* rows, const float* w, const float* b, float eps, T* out, int width) {
+  __shared__ float red[8];
+  griddep_wait();
+  const int src = rows ? rows[blockIdx.x] : int(blockIdx.x);
+  const float* xr = x + size_t(src) * width;
+  float sum = 0.0f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) sum += xr[c];
+  const float mean = block_sum(sum, red) / float(width);
+  float ss = 0.0f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) ss = fmaf(xr[c] - mean, xr[c] - mean, ss);
+  const float f = 1.0f / sqrtf(block_sum(ss, red) / float(width) + eps);
+  for (int c = threadIdx.x; c < width; c += blockDim.x) out[size_t(blockIdx.x) * width + c] = to_act<T>(fmaf((xr[c] - mean) * f, w[c], b[c]));
 }
 
 // act[r, c] = gelu_tanh(gate[r, c]) * table[token[r], col + c], c < dim

@@ -61,6 +61,7 @@ struct mtx_layered {
   // MTX_NORM_PRE layers (they share h and xb with the parallel ones): the output gate of a recurrence whose gate is low-rank
   bool prenorm = false;
   int max_rec_gate = 0, max_rec_z = 0;
+  bool outlayer = false;  // MTX_NORM_OUT_LAYER layers
   float *rec_gate = nullptr, *rec_z = nullptr;
 };
 
@@ -143,14 +144,40 @@ __global__ void gate_up_bf16_kernel(const bf16* src, bf16* act, int ff, long lon
   }
 }
 
+// eight columns per thread: fp32 values of a bf16 projection, the columns [silu0, silu1) through silu and rounded to bf16 again
+__global__ void __launch_bounds__(256) bf16_cols_to_f32_kernel(const bf16* src, float* dst, int n, int silu0, int silu1, long long groups) {
+  griddep_wait();
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < groups; i += (long long)gridDim.x * blockDim.x) {
+    const uint4 q = *reinterpret_cast<const uint4*>(src + i * 8);
+    const int c0 = int((i * 8) % n);
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[e]));
+      v[2 * e] = f.x;
+      v[2 * e + 1] = f.y;
+    }
+    if (c0 + 8 > silu0 && c0 < silu1) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e)
+        if (c0 + e >= silu0 && c0 + e < silu1) v[e] = __bfloat162float(__float2bfloat16_rn(silu_gate_f(v[e], 1.0f)));
+    }
+    *reinterpret_cast<float4*>(dst + i * 8) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(dst + i * 8 + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+
 // out (fp32, or the gated activation) = EPI(a[rows, k] . w[n, k]^T)
 template <typename T, int EPI>
 int run_linear(mtx_layered* e, const void* a, const void* w, const float* bias, float* out, void* act, int rows, int n, int k, cudaStream_t st,
-               float limit = 0.0f, long long ldo = 0) {
+               float limit = 0.0f, long long ldo = 0, int silu0 = 0, int silu1 = 0) {
   if (rows <= 0) return MTX_OK;
   LinArgs<T> p;
   memset(&p, 0, sizeof(p));
   p.limit = limit;
+  p.silu0 = silu0;
+  p.silu1 = silu1;
   p.a = static_cast<const T*>(a);
   p.w = static_cast<const T*>(w);
   p.bias = bias;
@@ -166,16 +193,36 @@ int run_linear(mtx_layered* e, const void* a, const void* w, const float* bias, 
   else return launch(linear_mma_kernel<EPI>, grid, dim3(kLinThreads), 0, st, p);
 }
 
-// (relu2: max(., 0)^2; act has the row pitch ldo)
-__global__ void act_bf16_kernel(const bf16* src, bf16* act, int n, long long ldo, long long total, int relu2) {
+// (kind LIN_RELU2: max(., 0)^2; LIN_GELU: gelu_tanh(.); act has the row pitch ldo)
+__device__ __forceinline__ float act_of_kind(float v, int kind) {
+  if (kind == LIN_GELU) return gelu_tanh_f(v);
+  if (kind == LIN_RELU2) {
+    v = fmaxf(v, 0.0f);
+    v *= v;
+  }
+  return v;
+}
+
+// the same with eight columns per thread (n and ldo multiples of 8)
+__global__ void __launch_bounds__(256) act8_bf16_kernel(const bf16* src, bf16* act, int n, long long ldo, long long groups, int kind) {
+  griddep_wait();
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < groups; i += (long long)gridDim.x * blockDim.x) {
+    const uint4 q = *reinterpret_cast<const uint4*>(src + i * 8);
+    uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[e]));
+      const __nv_bfloat162 o = __floats2bfloat162_rn(act_of_kind(f.x, kind), act_of_kind(f.y, kind));
+      w[e] = *reinterpret_cast<const uint32_t*>(&o);
+    }
+    *reinterpret_cast<uint4*>(act + (i * 8 / n) * ldo + (i * 8) % n) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+}
+
+__global__ void act_bf16_kernel(const bf16* src, bf16* act, int n, long long ldo, long long total, int kind) {
   griddep_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-    float v = __bfloat162float(src[i]);
-    if (relu2) {
-      v = fmaxf(v, 0.0f);
-      v *= v;
-    }
-    act[(i / n) * ldo + i % n] = __float2bfloat16_rn(v);
+    act[(i / n) * ldo + i % n] = __float2bfloat16_rn(act_of_kind(__bfloat162float(src[i]), kind));
   }
 }
 
@@ -196,14 +243,20 @@ int run_umma_raw(mtx_layered* e, const void* a, const void* w, int rows, int n, 
 // ... then the epilogue as a row kernel
 template <int EPI>
 int run_linear_umma(mtx_layered* e, const void* a, const void* w, const float* bias, float* out, void* act, int rows, int n, int k, cudaStream_t st,
-                    float limit = 0.0f, long long ldo = 0) {
+                    float limit = 0.0f, long long ldo = 0, int silu0 = 0, int silu1 = 0) {
   MTX_TRY(run_umma_raw(e, a, w, rows, n, k, st));
   const bf16* tmp = static_cast<const bf16*>(e->obf);
   constexpr bool gated = EPI == LIN_GATED || EPI == LIN_GATED_CLAMP;
   const long long total = (long long)rows * (gated ? n / 2 : n);
   const int blocks = int((total + 255) / 256 < 148 * 8 ? (total + 255) / 256 : 148 * 8);
-  if (EPI == LIN_ACT || EPI == LIN_RELU2)
-    return launch(act_bf16_kernel, dim3(blocks), dim3(256), 0, st, tmp, static_cast<bf16*>(act), n, ldo > 0 ? ldo : (long long)n, total, EPI == LIN_RELU2 ? 1 : 0);
+  const long long groups = total / 8;  // (n is a multiple of 128)
+  const int blocks8 = int((groups + 255) / 256 < 148 * 8 ? (groups + 255) / 256 : 148 * 8);
+  if (EPI == LIN_SILU_COLS) return launch(bf16_cols_to_f32_kernel, dim3(blocks8), dim3(256), 0, st, tmp, out, n, silu0, silu1, groups);
+  if (EPI == LIN_ACT || EPI == LIN_RELU2 || EPI == LIN_GELU) {
+    if (ldo <= 0) ldo = n;
+    if (ldo % 8 == 0 && (reinterpret_cast<uintptr_t>(act) & 15) == 0) return launch(act8_bf16_kernel, dim3(blocks8), dim3(256), 0, st, tmp, static_cast<bf16*>(act), n, ldo, groups, EPI);
+    return launch(act_bf16_kernel, dim3(blocks), dim3(256), 0, st, tmp, static_cast<bf16*>(act), n, ldo, total, EPI);
+  }
   if (gated)
     return launch(gate_up_bf16_kernel, dim3(blocks), dim3(256), 0, st, tmp, static_cast<bf16*>(act), n / 2, total, limit,
                   EPI == LIN_GATED_CLAMP ? (limit > 0.0f ? 1 : 2) : 0);
@@ -214,11 +267,11 @@ bool takes_umma(const mtx_layered* e, int rows, int n, int k) { return fits_umma
 
 template <typename T, int EPI>
 int linear(mtx_layered* e, const void* a, const void* w, const float* bias, float* out, void* act, int rows, int n, int k, cudaStream_t st,
-           float limit = 0.0f, long long ldo = 0) {
+           float limit = 0.0f, long long ldo = 0, int silu0 = 0, int silu1 = 0) {
   if constexpr (sizeof(T) == 2) {
-    if (takes_umma(e, rows, n, k)) return run_linear_umma<EPI>(e, a, w, bias, out, act, rows, n, k, st, limit, ldo);
+    if (takes_umma(e, rows, n, k)) return run_linear_umma<EPI>(e, a, w, bias, out, act, rows, n, k, st, limit, ldo, silu0, silu1);
   }
-  return run_linear<T, EPI>(e, a, w, bias, out, act, rows, n, k, st, limit, ldo);
+  return run_linear<T, EPI>(e, a, w, bias, out, act, rows, n, k, st, limit, ldo, silu0, silu1);
 }
 
 // `batches` products over the same rows whose operands lie side by side (linear_any.cuh, batched mode): batch z reads the columns
@@ -509,7 +562,7 @@ int window_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_t
 
 // Column layout of a composite mixer's input projection and of the activation its output projection reads.
 struct CompositeCols {
-  int aq = 0, ak = 0, av = -1, rq = 0, rk = 0, rv = 0, rg = 0, rx = 0, n = 0;
+  int aq = 0, ak = 0, av = -1, ag = 0, rq = 0, rk = 0, rv = 0, rg = 0, rx = 0, n = 0;
   int out_rec = 0, k_out = 0;
 };
 
@@ -527,6 +580,8 @@ CompositeCols composite_cols(const mtx_layer_desc& l) {
       cc.av = at;
       at += a.kv_heads * a.vdim;
     }
+    cc.ag = at;
+    if (a.value_gate) at += a.heads * a.vdim;
     cc.out_rec = a.heads * a.vdim;
   }
   if (r.kind != 0) {
@@ -539,7 +594,7 @@ CompositeCols composite_cols(const mtx_layer_desc& l) {
     cc.rg = at;
     at += r.heads * r.vdim;
     cc.rx = at;
-    at += r.kind == MTX_REC_GLA ? r.decay_rank : 2 * r.heads;
+    at += r.kind == MTX_REC_GLA ? r.decay_rank : (r.kind == MTX_REC_MLSTM ? 2 * r.heads : 0);
   }
   cc.n = at;
   cc.k_out = cc.out_rec + (r.kind != 0 ? r.heads * r.vdim : 0);
@@ -559,7 +614,7 @@ int launch_rec_scan_t(const RecScanArgs& ra, dim3 grid, dim3 block, size_t smem,
 template <int KIND, int CB, int SL>
 int launch_rec_scan_cb(const RecScanArgs& ra, int n_runs, cudaStream_t st) {
   const dim3 grid(n_runs, ra.heads, (ra.vdim + CB - 1) / CB), block(CB * SL);
-  const size_t smem = rec_scan_smem_bytes(ra.dim, CB, SL, ra.chunk, KIND == REC_DELTA ? 5 : 3);  // (the gated delta rule stages q, k, decays)
+  const size_t smem = rec_scan_smem_bytes(ra.dim, CB, SL, ra.chunk, rec_vectors(KIND));
   const int rpt = rec_rpt(ra.dim, SL);
   if (rpt == 4) return launch_rec_scan_t<KIND, 4, CB, SL>(ra, grid, block, smem, st);
   if (rpt == 8) return launch_rec_scan_t<KIND, 8, CB, SL>(ra, grid, block, smem, st);
@@ -577,7 +632,7 @@ int launch_rec_scan(mtx_layered* e, RecScanArgs& ra, int n_runs, int rows, cudaS
   const bool wide = (long long)n_runs * ra.heads * ((ra.vdim + 15) / 16) >= 2LL * e->num_sms;
   static const int force_sl = env_int("MTX_REC_SLICES", 0);
   const bool fine = force_sl ? force_sl == 16 : (!wide && ra.dim >= 64 && columns * 8 < 512LL * e->num_sms);
-  ra.chunk = rec_chunk_tokens(ra.dim, wide ? 16 : 8, fine ? 16 : 8, rows == n_runs, KIND == REC_DELTA ? 5 : 3);
+  ra.chunk = rec_chunk_tokens(ra.dim, wide ? 16 : 8, fine ? 16 : 8, rows == n_runs, rec_vectors(KIND));
   if (fine && ra.dim >= 16) return launch_rec_scan_cb<KIND, 8, 16>(ra, n_runs, st);
   return wide ? launch_rec_scan_cb<KIND, 16, 8>(ra, n_runs, st) : launch_rec_scan_cb<KIND, 8, 8>(ra, n_runs, st);
 }
@@ -815,6 +870,53 @@ int run_softmax_attention(mtx_layered* e, SoftmaxAttnArgs<T>& sa, const mtx_ragg
   return MTX_OK;
 }
 
+// A routed feed-forward of the rows `xa` up to its experts' outputs: router, choice, sort, the chosen experts' products into e->moe_y (slot
+// e->moe_slot of every (row, choice)), the shared expert's product into e->y, or -- shared_bf16 given and the tcgen05 projection
+// taken -- left as bf16 in e->obf (*shared_bf16 points there, else it is null).
+template <typename T>
+int routed_experts(mtx_layered* e, const mtx_moe_desc& m, const T* xa, int rows, cudaStream_t st, const bf16** shared_bf16 = nullptr) {
+  const int E = e->cfg.width, entries = rows * m.top;
+  const int n_all = m.experts + m.identity, ld = n_all + (m.shared_gate ? 1 : 0);  // router outputs; rows of the router's matrix
+  const float limit = m.act_silu ? 0.0f : m.limit, shared_limit = m.act_silu ? 0.0f : m.shared_limit;
+  if (ld <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, xa, static_cast<const T*>(m.w_router), m.router_bias, e->moe_logits, ld, E));
+  // (more experts: the any-shape kernel, whose result is fp32; the tcgen05 projection would round it)
+  else if (m.router_bias) MTX_TRY((run_linear<T, LIN_BIAS>(e, xa, m.w_router, m.router_bias, e->moe_logits, nullptr, rows, ld, E, st)));
+  else MTX_TRY((run_linear<T, LIN_PLAIN>(e, xa, m.w_router, nullptr, e->moe_logits, nullptr, rows, ld, E, st)));
+  MoeRouteArgs ra;
+  memset(&ra, 0, sizeof(ra));
+  ra.logits = e->moe_logits;
+  ra.ld = ld;
+  ra.correction = m.correction;
+  ra.chosen = e->moe_chosen;
+  ra.weight = e->moe_weight;
+  ra.experts = n_all;
+  ra.top = m.top;
+  ra.groups = m.groups > 0 ? m.groups : 1;
+  ra.keep = m.keep_groups > 0 ? m.keep_groups : 1;
+  ra.groups_max = m.groups_max;
+  ra.softmax = m.score_softmax;
+  ra.plain = m.plain_weights;
+  ra.chosen_softmax = m.chosen_softmax;
+  MTX_TRY(launch(moe_route_kernel, dim3(rows), dim3(32), sizeof(float) * (2 * n_all + ra.groups), st, ra));
+  // (identity experts get slot ranges behind the others': no product reads them)
+  MTX_TRY(launch(moe_sort_kernel, dim3(1), dim3(1024), sizeof(int) * (2 * n_all + 1), st, (const int*)e->moe_chosen, entries, m.top, n_all, e->moe_off, e->moe_slot,
+                 e->moe_row));
+  MTX_TRY((linear_grouped<T, LIN_GATED_CLAMP>(xa, e->moe_row, m.w_gate_up, (long long)2 * m.ff * E, e->moe_off, m.experts, nullptr, e->moe_act, entries, 2 * m.ff,
+                                              E, limit, st)));
+  MTX_TRY((linear_grouped<T, LIN_PLAIN>(e->moe_act, nullptr, m.w_down, (long long)E * m.ff, e->moe_off, m.experts, e->moe_y, nullptr, entries, E, m.ff, 0.0f, st)));
+  if (shared_bf16) *shared_bf16 = nullptr;
+  if (m.shared_ff > 0) {
+    MTX_TRY((linear<T, LIN_GATED_CLAMP>(e, xa, m.shared_gate_up, nullptr, nullptr, e->act, rows, 2 * m.shared_ff, E, st, shared_limit)));
+    if (sizeof(T) == 2 && shared_bf16 && takes_umma(e, rows, E, m.shared_ff)) {
+      MTX_TRY(run_umma_raw(e, e->act, m.shared_down, rows, E, m.shared_ff, st));
+      *shared_bf16 = static_cast<const bf16*>(e->obf);
+    } else {
+      MTX_TRY((linear<T, LIN_PLAIN>(e, e->act, m.shared_down, nullptr, e->y, nullptr, rows, E, m.shared_ff, st)));
+    }
+  }
+  return MTX_OK;
+}
+
 // a MTX_MIXER_COMPOSITE layer with MTX_NORM_SANDWICH norms; xa holds wnorm(x, norm1) on entry
 template <typename T>
 int composite_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_t st) {
@@ -940,30 +1042,7 @@ int composite_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStrea
   if (!has_ff) return MTX_OK;
   if (l.ff_kind == MTX_FF_MOE) {
     const mtx_moe_desc& m = l.moe;
-    const int entries = rows * m.top;
-    if (m.experts <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, (const T*)xa, static_cast<const T*>(m.w_router), (const float*)nullptr, e->moe_logits, m.experts, E));
-    else MTX_TRY((linear<T, LIN_PLAIN>(e, xa, m.w_router, nullptr, e->moe_logits, nullptr, rows, m.experts, E, st)));
-    MoeRouteArgs ra;
-    memset(&ra, 0, sizeof(ra));
-    ra.logits = e->moe_logits;
-    ra.correction = m.correction;
-    ra.chosen = e->moe_chosen;
-    ra.weight = e->moe_weight;
-    ra.experts = m.experts;
-    ra.top = m.top;
-    ra.groups = m.groups;
-    ra.keep = m.keep_groups;
-    MTX_TRY(launch(moe_route_kernel, dim3(rows), dim3(32), sizeof(float) * (2 * m.experts + m.groups), st, ra));
-    MTX_TRY(launch(moe_sort_kernel, dim3(1), dim3(1024), sizeof(int) * (2 * m.experts + 1), st, (const int*)e->moe_chosen, entries, m.top, m.experts,
-                   e->moe_off, e->moe_slot, e->moe_row));
-    MTX_TRY((linear_grouped<T, LIN_GATED_CLAMP>(xa, e->moe_row, m.w_gate_up, (long long)2 * m.ff * E, e->moe_off, m.experts, nullptr, e->moe_act, entries,
-                                                2 * m.ff, E, m.limit, st)));
-    MTX_TRY((linear_grouped<T, LIN_PLAIN>(e->moe_act, nullptr, m.w_down, (long long)E * m.ff, e->moe_off, m.experts, e->moe_y, nullptr, entries, E, m.ff,
-                                          0.0f, st)));
-    if (m.shared_ff > 0) {
-      MTX_TRY((linear<T, LIN_GATED_CLAMP>(e, xa, m.shared_gate_up, nullptr, nullptr, e->act, rows, 2 * m.shared_ff, E, st, m.shared_limit)));
-      MTX_TRY((linear<T, LIN_PLAIN>(e, e->act, m.shared_down, nullptr, e->y, nullptr, rows, E, m.shared_ff, st)));
-    }
+    MTX_TRY(routed_experts<T>(e, m, xa, rows, st));
     MTX_TRY(launch(moe_combine_kernel, dim3(rows), dim3(256), 0, st, (const float*)e->moe_y, (const int*)e->moe_slot, (const float*)e->moe_weight, m.top, E,
                    m.shared_ff > 0 ? 1 : 0, e->y));
   } else {
@@ -1578,36 +1657,7 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
   const bool has_ff = m.experts > 0, has_side = l.side_dim > 0;
   if (has_ff) {
     MTX_TRY(pre_norm_step<T>(e, e->y, nullptr, nullptr, false, -1, l.norm2, b, st));  // x += mixer; xa = unit(x) * norm2
-    const int entries = rows * m.top;
-    const float limit = m.act_silu ? 0.0f : m.limit, shared_limit = m.act_silu ? 0.0f : m.shared_limit;
-    if (m.experts <= 64) MTX_TRY(launch(moe_router_kernel<T>, dim3(rows), dim3(256), 0, st, (const T*)xa, static_cast<const T*>(m.w_router), m.router_bias, e->moe_logits, m.experts, E));
-    // (more experts: the any-shape kernel, whose result is fp32; the tcgen05 projection would round it)
-    else if (m.router_bias) MTX_TRY((run_linear<T, LIN_BIAS>(e, xa, m.w_router, m.router_bias, e->moe_logits, nullptr, rows, m.experts, E, st)));
-    else MTX_TRY((run_linear<T, LIN_PLAIN>(e, xa, m.w_router, nullptr, e->moe_logits, nullptr, rows, m.experts, E, st)));
-    MoeRouteArgs ra;
-    memset(&ra, 0, sizeof(ra));
-    ra.logits = e->moe_logits;
-    ra.correction = m.correction;
-    ra.chosen = e->moe_chosen;
-    ra.weight = e->moe_weight;
-    ra.experts = m.experts;
-    ra.top = m.top;
-    ra.groups = m.groups > 0 ? m.groups : 1;
-    ra.keep = m.keep_groups > 0 ? m.keep_groups : 1;
-    ra.softmax = m.score_softmax;
-    ra.plain = m.plain_weights;
-    ra.chosen_softmax = m.chosen_softmax;
-    MTX_TRY(launch(moe_route_kernel, dim3(rows), dim3(32), sizeof(float) * (2 * m.experts + ra.groups), st, ra));
-    MTX_TRY(launch(moe_sort_kernel, dim3(1), dim3(1024), sizeof(int) * (2 * m.experts + 1), st, (const int*)e->moe_chosen, entries, m.top, m.experts,
-                   e->moe_off, e->moe_slot, e->moe_row));
-    MTX_TRY((linear_grouped<T, LIN_GATED_CLAMP>(xa, e->moe_row, m.w_gate_up, (long long)2 * m.ff * E, e->moe_off, m.experts, nullptr, e->moe_act, entries,
-                                                2 * m.ff, E, limit, st)));
-    MTX_TRY((linear_grouped<T, LIN_PLAIN>(e->moe_act, nullptr, m.w_down, (long long)E * m.ff, e->moe_off, m.experts, e->moe_y, nullptr, entries, E, m.ff,
-                                          0.0f, st)));
-    if (m.shared_ff > 0) {
-      MTX_TRY((linear<T, LIN_GATED_CLAMP>(e, xa, m.shared_gate_up, nullptr, nullptr, e->act, rows, 2 * m.shared_ff, E, st, shared_limit)));
-      MTX_TRY((linear<T, LIN_PLAIN>(e, e->act, m.shared_down, nullptr, e->y, nullptr, rows, E, m.shared_ff, st)));
-    }
+    MTX_TRY(routed_experts<T>(e, m, xa, rows, st));
     MTX_TRY(launch(moe_combine_kernel, dim3(rows), dim3(256), 0, st, (const float*)e->moe_y, (const int*)e->moe_slot, (const float*)e->moe_weight, m.top, E,
                    m.shared_ff > 0 ? 1 : 0, e->y));
   }
@@ -1624,6 +1674,156 @@ int prenorm_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_
   return pre_norm_step<T>(e, e->y, l.side_norm, nullptr, false, li + 1, nullptr, b, st);  // x += unit(y) * side_norm; the next layer's norm
 }
 
+// MTX_NORM_OUT_LAYER: x += ln(y) * w + b and its copy in the matmul dtype; `a` names what y is
+template <typename T>
+int out_layer_norm(mtx_layered* e, OutLayerNormArgs a, const float* w, const float* b, int rows, cudaStream_t st) {
+  a.w = w;
+  a.b = b;
+  a.x = e->x;
+  a.eps = e->cfg.eps;
+  a.width = e->cfg.width;
+  if (a.width % 4 == 0) return launch(out_layer_norm_kernel<T, 4>, dim3(rows), dim3(256), 0, st, a, static_cast<T*>(e->xa));
+  return launch(out_layer_norm_kernel<T, 1>, dim3(rows), dim3(256), 0, st, a, static_cast<T*>(e->xa));
+}
+
+// ... of the projection a . w^T
+template <typename T>
+int project_out_layer_norm(mtx_layered* e, const void* a, const void* w, int k, const float* nw, const float* nb, int rows, cudaStream_t st) {
+  OutLayerNormArgs oa;
+  memset(&oa, 0, sizeof(oa));
+  if (sizeof(T) == 2 && takes_umma(e, rows, e->cfg.width, k)) {
+    MTX_TRY(run_umma_raw(e, a, w, rows, e->cfg.width, k, st));
+    oa.y_bf16 = static_cast<const bf16*>(e->obf);
+  } else {
+    MTX_TRY((linear<T, LIN_PLAIN>(e, a, w, nullptr, e->y, nullptr, rows, e->cfg.width, k, st)));
+    oa.y = e->y;
+  }
+  return out_layer_norm<T>(e, oa, nw, nb, rows, st);
+}
+
+// a MTX_NORM_OUT_LAYER layer: both sublayers read x itself (xa = x in the matmul dtype)
+template <typename T>
+int outlayer_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_t st) {
+  const mtx_layered_config& c = e->cfg;
+  const mtx_layer_desc& l = e->layers[li];
+  const int rows = b.rows, E = c.width, n_in = l.n_in;
+  T* xa = static_cast<T*>(e->xa);
+  T* mix = static_cast<T*>(e->attn);  // [rows, k_out]: the attention's heads, then the recurrence's
+  const CompositeCols cc = composite_cols(l);
+  const mtx_softmax_attn_desc& a = l.attn;
+  const mtx_recurrent_desc& r = l.rec;
+  // (the recurrence's q, k and v are next to one another: silu on the way)
+  MTX_TRY((linear<T, LIN_SILU_COLS>(e, xa, l.w_in, nullptr, e->qkv, nullptr, rows, n_in, E, st, 0.0f, 0, cc.rq, r.kind != 0 ? cc.rg : cc.rq)));
+  if (a.heads > 0) {
+    QkPrepareArgs<T> qa;
+    memset(&qa, 0, sizeof(qa));
+    qa.proj = e->qkv;
+    qa.ld = n_in;
+    qa.q_col = cc.aq;
+    qa.k_col = cc.ak;
+    qa.v_col = cc.av;
+    qa.q_norm = a.q_norm;
+    qa.k_norm = a.k_norm;
+    qa.rot_freq = a.rot_freq;
+    qa.q_out = static_cast<T*>(e->q);
+    qa.k_pages = static_cast<T*>(a.k_pages);
+    qa.v_pages = static_cast<T*>(a.v_pages);
+    qa.group = b.group;
+    qa.pos = b.pos;
+    qa.page_map = b.page_map;
+    qa.heads = a.heads;
+    qa.kv_heads = a.kv_heads;
+    qa.dim = a.dim;
+    qa.vdim = a.vdim;
+    qa.rot_dims = a.rot_dims;
+    qa.rot_half = a.rot_half;
+    qa.num_pages = c.num_pages;
+    qa.tokens_per_page = c.tokens_per_page;
+    qa.max_pages = c.max_pages_per_group;
+    qa.eps = c.eps;
+    MTX_TRY(launch(qk_prepare_append_kernel<T>, dim3(rows), dim3(256), 0, st, qa));
+    SoftmaxAttnArgs<T> sa = attention_args<T>(c, b);
+    sa.q = static_cast<const T*>(e->q);
+    sa.out = mix;
+    sa.ld_out = cc.k_out;
+    sa.k_pages = static_cast<const T*>(a.k_pages);
+    sa.v_pages = static_cast<const T*>(a.v_pages);
+    sa.heads = a.heads;
+    sa.kv_heads = a.kv_heads;
+    sa.dim = a.dim;
+    sa.vdim = a.vdim;
+    sa.window = a.window;
+    sa.keep_first = a.keep_first;
+    sa.scale = a.scale;
+    sa.out_scale = a.out_scale;
+    sa.sink = a.sink;
+    sa.gate = a.value_gate ? e->qkv + cc.ag : nullptr;
+    sa.ld_gate = n_in;
+    sa.value_gate = a.value_gate;
+    MTX_TRY(run_softmax_attention<T>(e, sa, b, st));
+  }
+  if (r.kind != 0) {
+    RecScanArgs ra;
+    memset(&ra, 0, sizeof(ra));
+    ra.proj = e->qkv;
+    ra.ld = n_in;
+    ra.q_col = cc.rq;
+    ra.k_col = cc.rk;
+    ra.v_col = cc.rv;
+    ra.o = e->rec_o;
+    ra.state_s = r.state_s;
+    ra.head_decay = r.head_decay;
+    ra.run_row0 = b.run_row0;
+    ra.group = b.group;
+    ra.pos = b.pos;
+    ra.heads = r.heads;
+    ra.dim = r.dim;
+    ra.vdim = r.vdim;
+    ra.q_scale = r.q_scale;
+    ra.vec4 = (n_in % 4 == 0 && cc.rq % 4 == 0 && r.dim % 4 == 0 && r.vdim % 4 == 0) ? 1 : 0;
+    MTX_TRY(launch_rec_scan<REC_DECAY>(e, ra, b.n_runs, rows, st));
+    RecOutArgs<T> oa;
+    memset(&oa, 0, sizeof(oa));
+    oa.o = e->rec_o;
+    oa.proj = e->qkv;
+    oa.ld = n_in;
+    oa.g_col = cc.rg;
+    oa.weight = r.out_norm;
+    oa.out = mix;
+    oa.ld_out = cc.k_out;
+    oa.out_col = cc.out_rec;
+    oa.heads = r.heads;
+    oa.vdim = r.vdim;
+    oa.gate_silu = r.gate_silu;
+    oa.norm_whole = r.norm_whole;
+    oa.eps = c.eps;
+    oa.out_scale = r.out_scale;
+    MTX_TRY(launch(recurrent_out_kernel<T>, dim3(rows), dim3(256), 0, st, oa));
+  }
+  MTX_TRY(project_out_layer_norm<T>(e, mix, l.wo, cc.k_out, l.norm1, l.norm1b, rows, st));
+  if (l.ff_kind == MTX_FF_MOE) {
+    const mtx_moe_desc& m = l.moe;
+    OutLayerNormArgs oa;
+    memset(&oa, 0, sizeof(oa));
+    MTX_TRY(routed_experts<T>(e, m, xa, rows, st, &oa.y_bf16));
+    if (m.shared_ff > 0 && !oa.y_bf16) oa.y = e->y;
+    if (m.shared_gate) oa.shared_gate = e->moe_logits + m.experts + m.identity;
+    oa.ld_gate = m.experts + m.identity + 1;
+    oa.expert_y = e->moe_y;
+    oa.slot_of = e->moe_slot;
+    oa.chosen = e->moe_chosen;
+    oa.weight = e->moe_weight;
+    oa.top = m.top;
+    oa.experts = m.experts;
+    return out_layer_norm<T>(e, oa, l.norm2, l.norm2b, rows, st);
+  }
+  if (l.ff > 0) {
+    MTX_TRY((linear<T, LIN_GELU>(e, xa, l.w_gate_up, nullptr, nullptr, e->act, rows, l.ff, E, st)));
+    return project_out_layer_norm<T>(e, e->act, l.w_down, l.ff, l.norm2, l.norm2b, rows, st);
+  }
+  return MTX_OK;
+}
+
 template <typename T>
 int step_typed(mtx_layered* e, const mtx_ragged_batch& b, cudaStream_t st) {
   const mtx_layered_config& c = e->cfg;
@@ -1635,14 +1835,16 @@ int step_typed(mtx_layered* e, const mtx_ragged_batch& b, cudaStream_t st) {
   if (e->parallel) MTX_TRY(group_norm_step<T>(e, nullptr, 0.0f, 0, b, st));                         // layer 0's norm
   if (e->prenorm) MTX_TRY(pre_norm_step<T>(e, nullptr, nullptr, c.embed_norm, false, 0, nullptr, b, st));  // the embedding's norm, layer 0's norm
   for (int li = 0; li < c.num_layers; ++li) {
-    if (e->layers[li].norm_style == MTX_NORM_PRE) MTX_TRY(prenorm_layer<T>(e, li, b, st));
+    if (e->layers[li].norm_style == MTX_NORM_OUT_LAYER) MTX_TRY(outlayer_layer<T>(e, li, b, st));
+    else if (e->layers[li].norm_style == MTX_NORM_PRE) MTX_TRY(prenorm_layer<T>(e, li, b, st));
     else if (e->layers[li].norm_style == MTX_NORM_PARALLEL) MTX_TRY(parallel_layer<T>(e, li, b, st));
     else if (e->layers[li].mixer == MTX_MIXER_COMPOSITE) MTX_TRY(composite_layer<T>(e, li, b, st));
     else MTX_TRY(window_layer<T>(e, li, b, st));
   }
   if (b.n_want > 0) {
     T* wn = static_cast<T*>(e->wanted);
-    if (e->parallel || e->prenorm)
+    if (e->outlayer) MTX_TRY(launch(layer_norm_rows_kernel<T>, dim3(b.n_want), dim3(256), 0, st, (const float*)e->x, b.want_rows, c.final_norm, c.final_norm_b, c.eps, wn, E));
+    else if (e->parallel || e->prenorm)
       MTX_TRY(launch(group_norm_rows_kernel<T>, dim3(b.n_want), dim3(256), 0, st, (const float*)e->x, b.want_rows, c.final_norm, c.eps, wn, E,
                      e->prenorm ? 1 : c.norm_groups));
     else if (c.final_norm) MTX_TRY(launch(weighted_norm_rows_kernel<T>, dim3(b.n_want), dim3(256), 0, st, (const float*)e->x, b.want_rows, c.final_norm, c.eps, wn, E));
@@ -1860,6 +2062,67 @@ int check_prenorm(mtx_layered* e, int i) {
   return MTX_OK;
 }
 
+// validation and workspace sizes of a routed feed-forward with identity experts and groups scored by their largest choice score
+int check_routed(mtx_layered* e, int i) {
+  const mtx_moe_desc& m = e->layers[i].moe;
+  const int n_all = m.experts + m.identity, groups = m.groups > 0 ? m.groups : 1, keep = m.keep_groups > 0 ? m.keep_groups : 1;
+  if (m.experts < 1 || m.identity < 0 || m.top < 1 || n_all % groups != 0 || keep > groups || m.ff < 1 || keep * (n_all / groups) < m.top)
+    return fail(MTX_ERR_ARG, "layer %d: bad expert / identity / top / groups / ff", i);
+  if (n_all > 4096) return fail(MTX_ERR_UNSUPPORTED, "layer %d: more than 4096 experts", i);
+  if (!m.w_router || !m.w_gate_up || !m.w_down || (m.shared_ff > 0 && (!m.shared_gate_up || !m.shared_down))) return fail(MTX_ERR_ARG, "layer %d: an expert weight is missing", i);
+  if (m.shared_gate && (m.shared_ff < 1 || m.router_bias)) return fail(MTX_ERR_UNSUPPORTED, "layer %d: a shared expert's gate without that expert, or with router biases", i);
+  if (m.top > e->max_moe_top) e->max_moe_top = m.top;
+  if (n_all + 1 > e->max_moe_experts) e->max_moe_experts = n_all + 1;
+  if (m.ff > e->max_moe_ff) e->max_moe_ff = m.ff;
+  if (m.shared_ff > e->max_ff) e->max_ff = m.shared_ff;
+  if (2 * m.shared_ff > e->max_nqkv) e->max_nqkv = 2 * m.shared_ff;
+  return MTX_OK;
+}
+
+// validation and workspace sizes of a MTX_NORM_OUT_LAYER layer
+int check_outlayer(mtx_layered* e, int i) {
+  const mtx_layer_desc& l = e->layers[i];
+  const mtx_softmax_attn_desc& a = l.attn;
+  const mtx_recurrent_desc& r = l.rec;
+  if (l.mixer != MTX_MIXER_COMPOSITE || l.latent.heads > 0 || (a.heads <= 0 && r.kind == 0))
+    return fail(MTX_ERR_UNSUPPORTED, "layer %d: a layer with layer norms on its outputs has a softmax attention and / or a recurrence", i);
+  if (!l.norm1 || !l.norm1b || !l.w_in || !l.wo) return fail(MTX_ERR_ARG, "layer %d: a norm vector or a projection is missing", i);
+  if (l.b_in || l.bo || l.conv1 || l.side_dim > 0 || l.add_embedding || l.add_vector)
+    return fail(MTX_ERR_UNSUPPORTED, "layer %d: biases, input convolutions, side inputs and pre-adds belong to other layer styles", i);
+  if (a.heads > 0) {
+    if (a.kv_heads < 1 || a.heads % a.kv_heads != 0 || a.dim < 1 || a.vdim < 1 || a.window < 0) return fail(MTX_ERR_ARG, "layer %d: bad attention geometry", i);
+    if (a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims & 1) || (a.rot_dims > 0 && !a.rot_freq)) return fail(MTX_ERR_ARG, "layer %d: bad rot_dims / rot_freq", i);
+    if (a.values_are_keys || a.head_gate || a.shared_kv || a.pool || a.slopes || a.softcap > 0.0f || a.norm_whole || a.chunk || a.maps > 1 || a.temp || a.talk)
+      return fail(MTX_ERR_UNSUPPORTED, "layer %d: an optional part of the attention that belongs to other layer styles", i);
+    if (a.keep_first < 0 || (a.keep_first > 0 && a.window < 1)) return fail(MTX_ERR_ARG, "layer %d: kept first tokens need a window", i);
+    if (!a.k_pages || !a.v_pages) return fail(MTX_ERR_ARG, "layer %d: a page pool is missing", i);
+    if (kSmaxRows * a.vdim > kSmaxThreads * kSmaxMaxAcc) return fail(MTX_ERR_UNSUPPORTED, "layer %d: vdim %d exceeds %d", i, a.vdim, kSmaxThreads * kSmaxMaxAcc / kSmaxRows);
+    if (softmax_attn_smem_bytes(a.dim, a.vdim) > 200 * 1024) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the attention's heads do not fit shared memory", i);
+    if (a.heads * a.dim > e->max_qdim) e->max_qdim = a.heads * a.dim;
+    if (a.heads > e->max_attn_heads) e->max_attn_heads = a.heads;
+  }
+  if (r.kind != 0) {
+    if (r.kind != MTX_REC_DECAY) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the recurrence beside layer norms on the outputs is the decayed sum", i);
+    if (r.heads < 1 || r.dim < 1 || r.vdim < 1 || r.dim > kRecSlices * 32) return fail(MTX_ERR_UNSUPPORTED, "layer %d: recurrence heads / dim (<= %d) / vdim", i, kRecSlices * 32);
+    if (!r.state_s || !r.out_norm || !r.head_decay) return fail(MTX_ERR_ARG, "layer %d: the recurrence's state, output norm or decays are missing", i);
+    if (r.heads * r.vdim > e->max_rec_o) e->max_rec_o = r.heads * r.vdim;
+  }
+  const CompositeCols cc = composite_cols(l);
+  if (l.n_in < cc.n) return fail(MTX_ERR_ARG, "layer %d: n_in = %d, the sub-mixers need %d projection rows", i, l.n_in, cc.n);
+  if (l.n_in > e->max_nqkv) e->max_nqkv = l.n_in;
+  if (cc.k_out > e->max_odim) e->max_odim = cc.k_out;
+  if (l.ff_kind == MTX_FF_MOE) {
+    if (l.moe.experts > 0 && (!l.norm2 || !l.norm2b)) return fail(MTX_ERR_ARG, "layer %d: a feed-forward norm vector is missing", i);
+    MTX_TRY(check_routed(e, i));
+  } else if (l.ff > 0) {
+    if (l.ff_kind != MTX_FF_GELU || !l.norm2 || !l.norm2b || !l.w_gate_up || !l.w_down) return fail(MTX_ERR_ARG, "layer %d: the feed-forward is down(gelu(up x)) with a norm of its own", i);
+    if (l.ff > e->max_nqkv) e->max_nqkv = l.ff;  // (a tcgen05 projection parks its bf16 result in a plane of max_nqkv columns)
+    if (l.ff > e->max_ff) e->max_ff = l.ff;
+  }
+  e->outlayer = true;
+  return MTX_OK;
+}
+
 }  // namespace
 
 extern "C" {
@@ -1877,8 +2140,8 @@ int mtx_layered_create(const mtx_layered_config* cfg, const mtx_layer_desc* laye
   for (int i = 0; i < c.num_layers; ++i) {
     const mtx_layer_desc& l = e->layers[i];
     int rc = MTX_OK;
-    if (l.norm_style == MTX_NORM_PARALLEL || l.norm_style == MTX_NORM_PRE || l.mixer == MTX_MIXER_COMPOSITE) {
-      rc = l.norm_style == MTX_NORM_PRE ? check_prenorm(e, i) : (l.norm_style == MTX_NORM_PARALLEL ? check_parallel(e, i) : check_composite(e, i));
+    if (l.norm_style == MTX_NORM_PARALLEL || l.norm_style == MTX_NORM_PRE || l.norm_style == MTX_NORM_OUT_LAYER || l.mixer == MTX_MIXER_COMPOSITE) {
+      rc = l.norm_style == MTX_NORM_OUT_LAYER ? check_outlayer(e, i) : l.norm_style == MTX_NORM_PRE ? check_prenorm(e, i) : (l.norm_style == MTX_NORM_PARALLEL ? check_parallel(e, i) : check_composite(e, i));
       if (rc != MTX_OK) {
         delete e;
         return rc;
@@ -1930,6 +2193,19 @@ int mtx_layered_create(const mtx_layered_config* cfg, const mtx_layer_desc* laye
       delete e;
       return fail(MTX_ERR_UNSUPPORTED, "layer %d: all layers of a model share one norm style", i);
     }
+  for (int i = 0; i < c.num_layers; ++i)
+    if ((e->layers[i].norm_style == MTX_NORM_OUT_LAYER) != e->outlayer) {
+      delete e;
+      return fail(MTX_ERR_UNSUPPORTED, "layer %d: all layers of a model share one norm style", i);
+    }
+  if (e->outlayer && (!c.final_norm || !c.final_norm_b)) {
+    delete e;
+    return fail(MTX_ERR_ARG, "a model with layer norms on its outputs has a final norm with weight and bias");
+  }
+  if (e->outlayer && c.width > 256 * kOutLnVec) {
+    delete e;
+    return fail(MTX_ERR_UNSUPPORTED, "width %d exceeds %d", c.width, 256 * kOutLnVec);
+  }
   if ((e->parallel || e->prenorm) && !c.final_norm) {
     delete e;
     return fail(MTX_ERR_ARG, "a model of parallel or pre-norm layers has a final norm weight");
@@ -2003,7 +2279,7 @@ int mtx_layered_step(mtx_layered* e, const mtx_ragged_batch* b, mtx_stream strea
   if (b->n_want < 0 || b->n_want > e->cfg.max_want) return fail(MTX_ERR_ARG, "n_want = %d outside [0, %d]", b->n_want, e->cfg.max_want);
   if (!b->token || !b->group || !b->pos || !b->page_map || (b->n_want > 0 && (!b->want_rows || !b->logits))) return fail(MTX_ERR_ARG, "null batch array");
   if (b->n_tiles < 0 || b->n_tiles > b->rows) return fail(MTX_ERR_ARG, "n_tiles = %d for %d rows", b->n_tiles, b->rows);
-  if ((e->sandwich || e->parallel || e->prenorm) && (b->n_tiles < 1 || !b->tile_row0 || b->n_runs < 1 || b->n_runs > b->rows || !b->run_row0))
+  if ((e->sandwich || e->parallel || e->prenorm || e->outlayer) && (b->n_tiles < 1 || !b->tile_row0 || b->n_runs < 1 || b->n_runs > b->rows || !b->run_row0))
     return fail(MTX_ERR_ARG, "this model needs the batch's query tiles and runs");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return e->cfg.float32 ? step_typed<float>(e, *b, st) : step_typed<bf16>(e, *b, st);

@@ -14,6 +14,8 @@
 //                             limit <= 0: act[r, f] = silu(acc[r, 2f]) * acc[r, 2f + 1], no limits
 //            LIN_ACT    act[r, c] = acc                  (in the matmul dtype, row pitch ldo: the input of another product)
 //            LIN_RELU2  act[r, c] = max(acc, 0)^2
+//            LIN_GELU   act[r, c] = gelu_tanh(acc)
+//            LIN_SILU_COLS  out = acc, the columns [silu0, silu1) through silu and rounded to the matmul dtype (fp32)
 //
 // Batched mode (batch_a != 0 or batch_o != 0; group_off null): blockIdx.z names one of several products over the same rows whose
 // operands lie side by side: `a` moves by batch_a columns, the weight by w_group_stride elements and the output by batch_o columns
@@ -30,7 +32,7 @@
 
 namespace mtx {
 
-enum { LIN_PLAIN = 0, LIN_BIAS = 1, LIN_GATED = 2, LIN_GATED_CLAMP = 3, LIN_ACT = 4, LIN_RELU2 = 5 };
+enum { LIN_PLAIN = 0, LIN_BIAS = 1, LIN_GATED = 2, LIN_GATED_CLAMP = 3, LIN_ACT = 4, LIN_RELU2 = 5, LIN_GELU = 6, LIN_SILU_COLS = 7 };
 
 template <typename T>
 struct LinArgs {
@@ -42,6 +44,7 @@ struct LinArgs {
   long long lda, ldo;
   int rows, n, k;
   float limit;             // LIN_GATED_CLAMP
+  int silu0, silu1;        // LIN_SILU_COLS
   const int* group_off;    // grouped mode: [groups + 1] slot ranges
   const int* a_row;        // grouped mode: [slots] row of `a` per slot, or null
   long long w_group_stride;  // grouped / batched mode: elements between two groups' weights
@@ -122,7 +125,11 @@ __device__ __forceinline__ void lin_store_pair(const LinArgs<T>& p, int r, int c
     p.act[size_t(r) * p.ldo + (c >> 1)] = to_act<T>(p.limit > 0.0f ? clamped_gate_f(v0, v1, p.limit) : silu_gate_f(v0, v1));
     return;
   }
-  if (EPI == LIN_ACT || EPI == LIN_RELU2) {
+  if (EPI == LIN_ACT || EPI == LIN_RELU2 || EPI == LIN_GELU) {
+    if (EPI == LIN_GELU) {
+      v0 = gelu_tanh_f(v0);
+      v1 = gelu_tanh_f(v1);
+    }
     if (EPI == LIN_RELU2) {
       v0 = fmaxf(v0, 0.0f);
       v1 = fmaxf(v1, 0.0f);
@@ -135,6 +142,10 @@ __device__ __forceinline__ void lin_store_pair(const LinArgs<T>& p, int r, int c
     return;
   }
   float* o = p.out + size_t(r) * p.ldo + c;
+  if (EPI == LIN_SILU_COLS) {
+    if (c >= p.silu0 && c < p.silu1) v0 = act_f32(to_act<T>(silu_gate_f(v0, 1.0f)));
+    if (c + 1 >= p.silu0 && c + 1 < p.silu1) v1 = act_f32(to_act<T>(silu_gate_f(v1, 1.0f)));
+  }
   if (EPI == LIN_BIAS) {
     v0 += p.bias[c];
     if (c + 1 < p.n) v1 += p.bias[c + 1];

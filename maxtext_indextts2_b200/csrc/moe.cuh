@@ -2,13 +2,15 @@
 //
 //   moe_router_kernel   per row: the router's logits (plus a bias), fp32 accumulation
 //   moe_route_kernel    per row: s = sigmoid(logits) (or, softmax set, the softmax over all experts); choice = s + correction; the experts of all but the keep_groups best groups
-//                       (a group's score = the sum of its two largest choice scores) are barred; the `top` largest remaining choice
+//                       (a group's score = the sum of its two largest choice scores, or, groups_max set, the largest) are barred; the `top` largest remaining choice
 //                       scores are chosen (the lower index wins a tie); weights = s of the chosen / (their sum + 1e-20), or, plain set, s of the
 //                       chosen as it is.  With chosen_softmax the experts are chosen by logit + correction and
 //                       the weights are the softmax over the chosen experts' logits.  fp32.
+//                       The last router outputs may be identity experts (their output is the row itself): `experts` counts them in.
 //   moe_sort_kernel     one CTA: counts the (row, choice) entries per expert, lays the experts' slot ranges side by side
 //                       (group_off), gives every entry a slot in its expert's range and records the row each slot reads.
 //   moe_combine_kernel  y[row] (+)= sum over the row's choices, in the order of the choices, of weight * expert output of its slot.
+//                       (layer_ops.cuh's out_layer_norm_kernel does the same inside the norm that follows, with identity experts.)
 #pragma once
 
 #include "common.cuh"
@@ -59,6 +61,8 @@ struct MoeRouteArgs {
   int* chosen;              // [rows, top]
   float* weight;            // [rows, top]
   int experts, top, groups, keep;
+  int ld;                   // row pitch of logits
+  int groups_max;           // 1: a group's score is its largest choice score
   int softmax;              // 1: s = softmax(logits) over all experts
   int plain;                // 1: weights = s of the chosen, not renormalised
   int chosen_softmax;       // 1: s = logits; weights = softmax over the chosen
@@ -74,15 +78,15 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const MoeRouteArgs a) {
   const int r = blockIdx.x, lane = threadIdx.x, E = a.experts, per = E / a.groups;
   float zmax = -INFINITY, zsum = 1.0f;
   if (a.softmax) {
-    for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, a.logits[size_t(r) * E + e]);
+    for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, a.logits[size_t(r) * a.ld + e]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) zmax = fmaxf(zmax, __shfl_xor_sync(0xffffffffu, zmax, o));
     zsum = 0.0f;
-    for (int e = lane; e < E; e += 32) zsum += expf(a.logits[size_t(r) * E + e] - zmax);
+    for (int e = lane; e < E; e += 32) zsum += expf(a.logits[size_t(r) * a.ld + e] - zmax);
     zsum = warp_sum(zsum);
   }
   for (int e = lane; e < E; e += 32) {
-    const float z = a.logits[size_t(r) * E + e];
+    const float z = a.logits[size_t(r) * a.ld + e];
     const float v = a.chosen_softmax ? z : a.softmax ? expf(z - zmax) / zsum : 1.0f / (1.0f + expf(-z));
     s[e] = v;
     c[e] = v + (a.correction ? a.correction[e] : 0.0f);
@@ -100,7 +104,7 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const MoeRouteArgs a) {
           b2 = v;
         }
       }
-      gs[g] = per >= 2 ? b1 + b2 : b1;
+      gs[g] = per >= 2 && !a.groups_max ? b1 + b2 : b1;
     }
     __syncwarp();
     for (int g = lane; g < a.groups; g += 32) {

@@ -163,14 +163,15 @@ __global__ void __launch_bounds__(KT == 16 ? 128 : 256, DV16 <= 8 && KT >= 32 ? 
       if (a.group[rb] != grp || a.pos[rb] != pa + (rb - ra)) break;
       rb = a.tile_row0[tb + 1];
     }
-    const int lo = smax_first(pa, a.window, a.chunk), last = pa + (rb - ra) - 1, n_key_tiles = (last - lo) / KT + 1;
+    const int lo = smax_first(pa, a.window, a.chunk), last = pa + (rb - ra) - 1, lead = a.keep_first < lo ? a.keep_first : lo, skip = lo - lead,
+              v_last = last - skip, n_key_tiles = v_last / KT + 1;  // virtual key indices: see softmax_attention.cuh
     const int* pages = a.page_map + size_t(grp) * a.max_pages;
     const bool mine = active && my_tile >= ta && my_tile < tb;
     int rows_next[RPT];  // cache rows of this thread's keys of the tile that is copied next
     auto find_rows = [&](int it) {
 #pragma unroll
       for (int q = 0; q < RPT; ++q) {
-        const int jn = lo + it * KT + ld_row + q * (NT / 8), j = jn < last ? jn : last;
+        const int vn = it * KT + ld_row + q * (NT / 8), v = vn < v_last ? vn : v_last, j = v < lead ? v : v + skip;
         const int pg = page_shift >= 0 ? (j >> page_shift) : j / tpp;
         rows_next[q] = pages[pg] * tpp + (j - pg * tpp);
       }
@@ -196,8 +197,8 @@ __global__ void __launch_bounds__(KT == 16 ? 128 : 256, DV16 <= 8 && KT >= 32 ? 
         cp_async_wait_pending(0);
       }
       __syncthreads();
-      const int j0 = lo + it * KT;
-      if (mine && j0 <= p_last && j0 + KT > lo_first) {
+      const int v0 = it * KT, j0 = v0 < lead ? v0 : v0 + skip, j_end = v0 + KT <= lead ? v0 + KT : v0 + KT + skip;
+      if (mine && j0 <= p_last && (j_end > lo_first || j0 < a.keep_first)) {
         const bf16* sk = stage0 + size_t(it & 1) * stage_elems;
         const bf16* sv = same_kv ? sk : sk + KT * KP;
         float s[KT / 8][4];
@@ -219,7 +220,7 @@ __global__ void __launch_bounds__(KT == 16 ? 128 : 256, DV16 <= 8 && KT >= 32 ? 
             mma_bf16_16816(s[nb + 1], qf, kf[2], kf[3]);
           }
         }
-        const bool every_key_seen = j0 + KT - 1 <= p0 && j0 >= lo_last;
+        const bool every_key_seen = v0 < lead ? v0 + KT <= lead : j_end - 1 <= p0 && j0 >= lo_last;
         float mx0 = -INFINITY, mx1 = -INFINITY;  // (of the raw products: the scale is positive)
         if (every_key_seen) {
 #pragma unroll
@@ -232,8 +233,8 @@ __global__ void __launch_bounds__(KT == 16 ? 128 : 256, DV16 <= 8 && KT >= 32 ? 
           for (int nb = 0; nb < KT / 8; ++nb) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              const int j = j0 + nb * 8 + 2 * t + (e & 1);
-              if (j > ((e & 2) ? pi1 : pi0) || j < ((e & 2) ? lo1 : lo0)) s[nb][e] = -INFINITY;
+              const int v = v0 + nb * 8 + 2 * t + (e & 1), j = v < lead ? v : v + skip;
+              if (j > ((e & 2) ? pi1 : pi0) || (j < ((e & 2) ? lo1 : lo0) && j >= a.keep_first)) s[nb][e] = -INFINITY;
             }
             mx0 = fmaxf(mx0, fmaxf(s[nb][0], s[nb][1]));
             mx1 = fmaxf(mx1, fmaxf(s[nb][2], s[nb][3]));
@@ -339,8 +340,15 @@ __global__ void __launch_bounds__(KT == 16 ? 128 : 256, DV16 <= 8 && KT >= 32 ? 
     return;
   }
   if (!active) return;
-  const float f0 = a.out_scale / l_run[0] * (g < nr ? smax_gate(a.gate, a.ld_gate, r0 + g, h) : 1.0f);
-  const float f1 = a.out_scale / l_run[1] * (g + 8 < nr ? smax_gate(a.gate, a.ld_gate, r0 + g + 8, h) : 1.0f);
+  const float f0 = a.out_scale / l_run[0] * (g < nr ? smax_gate(a, r0 + g, h) : 1.0f);
+  const float f1 = a.out_scale / l_run[1] * (g + 8 < nr ? smax_gate(a, r0 + g + 8, h) : 1.0f);
+  if (a.value_gate) {
+#pragma unroll
+    for (int nb = 0; nb < NB; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (nb * 8 + 2 * t < dv && g + (e & 2) * 4 < nr) o[nb][e] *= smax_value_gate(a, r0 + g + (e & 2) * 4, h, nb * 8 + 2 * t + (e & 1));
+  }
 #pragma unroll
   for (int nb = 0; nb < NB; ++nb) {
     const int col = nb * 8 + 2 * t;
@@ -422,7 +430,8 @@ __global__ void __launch_bounds__(128) multi_attention_decode_kernel(const Softm
   const char* const kbase = reinterpret_cast<const char*>(a.k_pages + (a.wide ? 0 : size_t(vgroup) * maps * pool_rows * d));
   const char* const vbase = reinterpret_cast<const char*>(a.v_pages + size_t(vh0) * pool_rows * dv);
   const int vals_here = n_vals < a.kv_heads - vh0 ? n_vals : a.kv_heads - vh0;  // (the last group may hold fewer value heads)
-  const int all_key_tiles = (pos - lo) / KT + 1, per = (all_key_tiles + a.splits - 1) / a.splits, tile_lo = int(blockIdx.z) * per;
+  const int lead = a.keep_first < lo ? a.keep_first : lo, skip = lo - lead, v_last = pos - skip;
+  const int all_key_tiles = v_last / KT + 1, per = (all_key_tiles + a.splits - 1) / a.splits, tile_lo = int(blockIdx.z) * per;
   int n_key_tiles = all_key_tiles - tile_lo < per ? all_key_tiles - tile_lo : per;
   if (n_key_tiles < 0) n_key_tiles = 0;
   // column hh of unit group s: its unit (-1: none) and, among the group's value heads, its value head
@@ -439,7 +448,7 @@ __global__ void __launch_bounds__(128) multi_attention_decode_kernel(const Softm
 #pragma unroll
     for (int q = 0; q < 4; ++q)
       if (q < ks_n) {
-        const int jn = lo + (tile_lo + it) * KT + ld_row + q * 16, j = jn < pos ? jn : pos;
+        const int vn = (tile_lo + it) * KT + ld_row + q * 16, v = vn < v_last ? vn : v_last, j = v < lead ? v : v + skip;
         const int pg = page_shift >= 0 ? (j >> page_shift) : j / tpp;
         rows_next[q] = pages[pg] * tpp + (j - pg * tpp);
       }
@@ -501,8 +510,8 @@ __global__ void __launch_bounds__(128) multi_attention_decode_kernel(const Softm
     __syncthreads();
     const bf16* sk = stage0 + size_t(it & 1) * stage_elems;
     const bf16* sv = same_kv ? sk : sk + KT * KP;
-    const int j0 = lo + (tile_lo + it) * KT + ks * 16;  // this warp's 16 keys
-    if (j0 <= pos) {
+    const int j0 = (tile_lo + it) * KT + ks * 16;  // this warp's 16 keys
+    if (j0 <= v_last) {
       float c[4] = {0.0f, 0.0f, 0.0f, 0.0f}, c2[4] = {0.0f, 0.0f, 0.0f, 0.0f};  // two chains
       const bf16* kb = sk + (ks * 16 + (lane & 15)) * KP + (lane >> 4) * 8;
       const bf16* qb = sQ + (set * 8 + (lane & 7)) * KP + (lane >> 3) * 8;  // (four 8-channel columns of the eight units per ldmatrix)
@@ -522,7 +531,7 @@ __global__ void __launch_bounds__(128) multi_attention_decode_kernel(const Softm
         mat_ldsm_x4(af, kb + k0);
         mma_bf16_16816(c, af, *reinterpret_cast<const uint32_t*>(q1), *reinterpret_cast<const uint32_t*>(q1 + 8));
       }
-      const bool sa = j0 + g <= pos, sb = j0 + g + 8 <= pos;  // (no tile starts before the first visible key)
+      const bool sa = j0 + g <= v_last, sb = j0 + g + 8 <= v_last;  // (every key of the walk up to its end is visible)
       c[0] = sa ? (c[0] + c2[0]) * mul : -INFINITY;
       c[1] = sa ? (c[1] + c2[1]) * mul : -INFINITY;
       c[2] = sb ? (c[2] + c2[2]) * mul : -INFINITY;
@@ -622,14 +631,14 @@ __global__ void __launch_bounds__(128) multi_attention_decode_kernel(const Softm
       a.part_ml[base * 2] = M * 0.6931471805599453f;  // (the merge kernels work with natural exponents)
       a.part_ml[base * 2 + 1] = L;
     }
-    const float f = partial ? 1.0f : a.out_scale / L * smax_gate(a.gate, a.ld_gate, row, u / maps);
+    const float f = partial ? 1.0f : a.out_scale / L * smax_gate(a, row, u / maps);
     for (int col = lane; col < dv; col += 32) {
       float acc = 0.0f;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
         if (i < ks_n) acc = fmaf(w[i], mo[((s * ks_n + i) * 8 + hh) * dvp + col], acc);
       if (partial) a.part_o[base * dv + col] = acc;
-      else a.out[size_t(row) * a.ld_out + u * dv + col] = __float2bfloat16_rn(acc * f);
+      else a.out[size_t(row) * a.ld_out + u * dv + col] = __float2bfloat16_rn(acc * f * smax_value_gate(a, row, u, col));
     }
   }
 }

@@ -10,6 +10,7 @@
 //   gated delta  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q   (the read-out sees the token's own write)
 //          q, k, v after a short causal convolution over time and silu; q, k unit vectors (q / k heads may serve several heads);
 //          g = exp(-exp(a_log) softplus(z + bias)) per head or per key channel; beta = sigmoid(.)
+//   decay  S <- c S + k v^T,  o = S^T q                             c one constant per head (lightning attention); q, k, v through silu
 //
 // A run (consecutive rows of one sequence) is walked in order from the group's state; a run that starts at position 0 starts
 // from zero instead, so a slot that is handed to another sequence needs no clearing.  Every value column of S is independent of
@@ -22,7 +23,7 @@
 //   lowrank_split_kernel       the inputs of the gated delta rule's low-rank decay and gate projections in the matmul dtype
 //   gdelta_prepare_kernel      per row: the gated delta rule's convolutions, silu, unit vectors, decays and write strengths
 //   recurrent_scan_kernel      the walk
-//   recurrent_out_kernel<T>    per row and head: o / rms(o) * weight * gate(g) * out_scale -> the activation of the output projection
+//   recurrent_out_kernel<T>    per row and head (or over all heads of the row together): o / rms(o) * weight * gate(g) * out_scale -> the activation of the output projection
 #pragma once
 
 #include "common.cuh"
@@ -31,7 +32,7 @@
 
 namespace mtx {
 
-enum { REC_GLA = 1, REC_MLSTM = 2, REC_DELTA = 3, REC_GDELTA = 4 };
+enum { REC_GLA = 1, REC_MLSTM = 2, REC_DELTA = 3, REC_GDELTA = 4, REC_DECAY = 5 };
 
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 
@@ -257,6 +258,7 @@ struct RecScanArgs {
   // strength the column beta_col + h of the plane `aux` with row pitch aux_ld
   int qk_rep, dec_col, beta_col;
   long long aux_ld;
+  const float* head_decay;  // REC_DECAY: [heads]
 };
 
 // A CTA owns CB value columns of one (run, head): thread (column jl, slice sl) keeps RPT key channels of its column of S in
@@ -265,6 +267,9 @@ struct RecScanArgs {
 // / v arrive in chunks of `chunk` tokens (a multiple of 4) through a four-stage cp.async ring; tokens are walked four at a time
 // so that the four read-outs' reductions overlap (the state update itself is the only chain from token to token).
 constexpr int kRecSlices = 8, kRecUnroll = 4;  // (kRecSlices: the default; short of CTAs, a column is cut into 16 slices: SL)
+
+// per-channel vectors of a staged token: q, k and the decays; the delta rule also u and a u; constant decays are not staged
+__host__ __device__ constexpr int rec_vectors(int kind) { return kind == REC_DELTA ? 5 : (kind == REC_DECAY ? 2 : 3); }
 
 // floats of one token in a stage: q, k, decays (8 * RPT channels each), then CB values, then 4 scalars (mLSTM: log input gate,
 // log forget gate; later keep, put, floor)
@@ -299,7 +304,7 @@ __device__ __forceinline__ void rec_cp_async_4(float* dst, const float* src) {
 template <int KIND, int RPT, int CB, int SL>
 __global__ void __launch_bounds__(CB * SL) recurrent_scan_kernel(const RecScanArgs a) {
   extern __shared__ __align__(16) float rec_smem[];
-  constexpr int NV = KIND == REC_DELTA ? 5 : 3;                                   // per-channel vectors of a staged token
+  constexpr int NV = rec_vectors(KIND);
   constexpr int NT = CB * SL, QP = SL * RPT, TF = NV * QP + CB + 4, GS = 4 * SL;  // GS: channels per group of float4s
   const int d = a.dim, dv = a.vdim, H = a.heads, TC = a.chunk;
   const int tid = threadIdx.x, jl = tid / SL, sl = tid % SL;
@@ -343,6 +348,7 @@ __global__ void __launch_bounds__(CB * SL) recurrent_scan_kernel(const RecScanAr
     if (KIND == REC_MLSTM) m = a.state_m[size_t(slot) * H + h];
   }
   const int n_chunks = (nr + TC - 1) / TC;
+  const float decay_h = KIND == REC_DECAY ? a.head_decay[h] : 1.0f;
 
   // stage <- chunk c: every element by a 4-byte cp.async (the projection's columns have no alignment to count on); the tail of
   // the last chunk and the key channels beyond dim are filled with values that leave the state alone (k = v = q = 0, decay 1)
@@ -476,7 +482,21 @@ __global__ void __launch_bounds__(CB * SL) recurrent_scan_kernel(const RecScanAr
         part[u] = 0.0f;
         npart[u] = 0.0f;
         floor_m[u] = 0.0f;
-        if (KIND == REC_GLA) {
+        if (KIND == REC_DECAY) {
+          const float c = t0 + t + u < nr ? decay_h : 1.0f;  // (the filled tail leaves the state alone)
+#pragma unroll
+          for (int i4 = 0; i4 < RPT; i4 += 4) {
+            const float4 k4 = *reinterpret_cast<const float4*>(k + i4 * SL), q4 = *reinterpret_cast<const float4*>(q + i4 * SL);
+            S[i4] = fmaf(c, S[i4], k4.x * v);
+            S[i4 + 1] = fmaf(c, S[i4 + 1], k4.y * v);
+            S[i4 + 2] = fmaf(c, S[i4 + 2], k4.z * v);
+            S[i4 + 3] = fmaf(c, S[i4 + 3], k4.w * v);
+            part[u] = fmaf(S[i4], q4.x, part[u]);
+            part[u] = fmaf(S[i4 + 1], q4.y, part[u]);
+            part[u] = fmaf(S[i4 + 2], q4.z, part[u]);
+            part[u] = fmaf(S[i4 + 3], q4.w, part[u]);
+          }
+        } else if (KIND == REC_GLA) {
           const float* al = k + QP;
 #pragma unroll
           for (int i4 = 0; i4 < RPT; i4 += 4) {
@@ -623,6 +643,7 @@ struct RecOutArgs {
   int out_col;
   int heads, vdim, gate_silu;
   float eps, out_scale;
+  int norm_whole;       // 1: one root mean square over all heads of the row
 };
 
 // one CTA per row, a warp per head
@@ -630,6 +651,20 @@ template <typename T>
 __global__ void __launch_bounds__(256) recurrent_out_kernel(const RecOutArgs<T> a) {
   griddep_wait();
   const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, dv = a.vdim;
+  if (a.norm_whole) {
+    __shared__ float red[8];
+    const int n = a.heads * dv;
+    const float* o = a.o + size_t(r) * n;
+    const float* gate = a.proj + size_t(r) * a.ld + a.g_col;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(o[c], o[c], ss);
+    const float inv = a.out_scale / sqrtf(block_sum(ss, red) / float(n) + a.eps);
+    for (int c = threadIdx.x; c < n; c += blockDim.x) {
+      const float g = gate[c], sig = 1.0f / (1.0f + expf(-g));
+      a.out[size_t(r) * a.ld_out + a.out_col + c] = to_act<T>(o[c] * inv * a.weight[c] * (a.gate_silu ? g * sig : sig));
+    }
+    return;
+  }
   for (int h = warp; h < a.heads; h += nw) {
     const float* o = a.o + size_t(r) * a.heads * dv + h * dv;
     float ss = 0.0f;

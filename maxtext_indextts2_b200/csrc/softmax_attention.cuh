@@ -22,6 +22,12 @@
 //
 // A chunk size instead of a window (chunk > 0): a query at i sees the keys j <= i of its own chunk, j / chunk == i / chunk.
 //
+// Kept first tokens (keep_first = F > 0, with a window): beside its window every query sees the keys j < F.  A work item's keys are
+// then walked by a virtual index v that closes the gap between the kept tokens and the window of its first row: v < lead is the key
+// v, v >= lead the key v + skip, with lead = min(F, lo) and skip = lo - lead (F = 0: v = j - lo).
+//
+// The gate is one number per head, or (value_gate) one per channel of the concatenated heads.
+//
 // Two optional shapes of the scores (multi_attention.cuh has their tensor-core kernels):
 //   * maps == 2: every query head and every key head holds two vectors (score maps) over the same values; unit u = 2 h + m is
 //     head h's map m and reads key head 2 g + m, value head g.  The units' unnormalised results go to part_o / part_ml, and
@@ -294,6 +300,8 @@ struct SoftmaxAttnArgs {
   const T* kp_pages;    // [G, num_pages, pool_slots, d]
   const T* vp_pages;    // [G, num_pages, pool_slots, dv]
   int chunk;            // > 0 (window == 0): a query sees its own chunk of `chunk` positions up to itself
+  int keep_first;       // > 0 (window > 0, pool == 0): every query also sees the first keep_first tokens
+  int value_gate;       // 1: gate is [rows, ld_gate] with H * dv columns, one per channel of the concatenated heads
   int maps, wide;       // see the head of this file (0: one map per head, a key head per value head)
   float diff_lambda, diff_scale, eps;  // maps == 2
 };
@@ -326,8 +334,14 @@ __device__ __forceinline__ float smax_softcap_scaled(float raw, float mul, float
   return fmaf(-2.0f * cap, smax_rcp(1.0f + smax_ex2(raw * mul)), cap);
 }
 
-__device__ __forceinline__ float smax_gate(const float* gate, long long ld, int row, int h) {
-  return gate ? 1.0f / (1.0f + expf(-gate[size_t(row) * ld + h])) : 1.0f;
+// the head's gate (1 with gates per channel), and the channel's (1 without)
+template <typename A>
+__device__ __forceinline__ float smax_gate(const A& a, int row, int h) {
+  return a.gate && !a.value_gate ? 1.0f / (1.0f + expf(-a.gate[size_t(row) * a.ld_gate + h])) : 1.0f;
+}
+template <typename A>
+__device__ __forceinline__ float smax_value_gate(const A& a, int row, int h, int c) {
+  return a.value_gate ? 1.0f / (1.0f + __expf(-a.gate[size_t(row) * a.ld_gate + h * a.vdim + c])) : 1.0f;
 }
 
 constexpr int kSmaxThreads = 256, kSmaxRows = 16, kSmaxKeys = 32;
@@ -373,18 +387,20 @@ __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(co
   for (int u = 0; u < kSmaxMaxAcc; ++u) acc[u] = 0.0f;
   const int* pages = a.page_map + size_t(grp) * a.max_pages;
   const int nb_last = smax_blocks_seen(p_last, a.window, a.pool);
-  // two segments of keys: the pooled blocks 0 .. nb_last - 1 (if any), then the tokens lo .. p_last
+  const int lead = a.keep_first < lo ? a.keep_first : lo, skip = lo - lead;  // virtual key indices: see the head of this file
+  auto key_of = [&](int v, bool pooled) { return pooled || v < lead ? v : v + skip; };
+  // two segments of keys: the pooled blocks 0 .. nb_last - 1 (if any), then the kept tokens and the tokens lo .. p_last
   for (int seg = nb_last > 0 ? 0 : 1; seg < 2; ++seg) {
   const bool pooled = seg == 0;
-  const int begin = pooled ? 0 : lo, end = pooled ? nb_last - 1 : p_last, tpp = pooled ? a.pool_slots : a.tokens_per_page;
+  const int end = pooled ? nb_last - 1 : p_last - skip, tpp = pooled ? a.pool_slots : a.tokens_per_page;
   const T* kpool = pooled ? a.kp_pages : a.k_pages;
   const T* vpool = pooled ? a.vp_pages : a.v_pages;
   const size_t head_rows = size_t(g) * a.num_pages * tpp, key_rows = size_t(kh) * a.num_pages * tpp;
-  for (int j0 = begin; j0 <= end; j0 += kSmaxKeys) {
+  for (int j0 = 0; j0 <= end; j0 += kSmaxKeys) {
     const int nk = end - j0 + 1 < kSmaxKeys ? end - j0 + 1 : kSmaxKeys;
     __syncthreads();
     for (int e = tid; e < nk * dv; e += kSmaxThreads) {
-      const int jj = e / dv, c = e % dv, j = j0 + jj;
+      const int jj = e / dv, c = e % dv, j = key_of(j0 + jj, pooled);
       const size_t row = head_rows + size_t(pages[j / tpp]) * tpp + j % tpp;
       sv[jj * dv + c] = act_f32(vpool[row * dv + c]);
     }
@@ -396,7 +412,7 @@ __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(co
       if (c0 > 0) __syncthreads();
       if (ds < d) load_q(c0, n);
       for (int e = tid; e < nk * n; e += kSmaxThreads) {
-        const int jj = e / n, c = e % n, j = j0 + jj;
+        const int jj = e / n, c = e % n, j = key_of(j0 + jj, pooled);
         const size_t row = key_rows + size_t(pages[j / tpp]) * tpp + j % tpp;
         sk[jj * (ds + 1) + c] = act_f32(kpool[row * d + c0 + c]);
       }
@@ -413,10 +429,10 @@ __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(co
     }
 #pragma unroll
     for (int w = 0; w < kSmaxRows * kSmaxKeys / kSmaxThreads; ++w) {
-      const int e = tid + w * kSmaxThreads, i = e / kSmaxKeys, jj = e % kSmaxKeys, j = j0 + jj, pi = p0 + i;
+      const int e = tid + w * kSmaxThreads, i = e / kSmaxKeys, jj = e % kSmaxKeys, j = key_of(j0 + jj, pooled), pi = p0 + i;
       if (i >= nr) continue;
       float s = -INFINITY;
-      const bool seen = pooled ? j < smax_blocks_seen(pi, a.window, a.pool) : (j <= pi && j >= smax_first(pi, a.window, a.chunk));
+      const bool seen = pooled ? j < smax_blocks_seen(pi, a.window, a.pool) : (j <= pi && (j >= smax_first(pi, a.window, a.chunk) || j < a.keep_first));
       if (jj < nk && seen) {
         s = sc[w];
         if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
@@ -470,7 +486,7 @@ __global__ void __launch_bounds__(kSmaxThreads) softmax_attention_rows_kernel(co
         }
         continue;
       }
-      a.out[size_t(r0 + i) * a.ld_out + h * dv + c] = to_act<T>(acc[u] * a.out_scale / s_sum[i] * smax_gate(a.gate, a.ld_gate, r0 + i, h));
+      a.out[size_t(r0 + i) * a.ld_out + h * dv + c] = to_act<T>(acc[u] * a.out_scale / s_sum[i] * smax_gate(a, r0 + i, h) * smax_value_gate(a, r0 + i, h, c));
     }
   }
 }
@@ -526,7 +542,8 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
   const int nb_last = smax_blocks_seen(p_last, a.window, a.pool), pool_tiles = (nb_last + KT - 1) / KT;
   const int pool_shift = (a.pool_slots & (a.pool_slots - 1)) == 0 && a.pool_slots > 0 ? __ffs(a.pool_slots) - 1 : -1;
   const size_t pool_head_rows = size_t(kvh) * a.num_pages * a.pool_slots;
-  const int all_key_tiles = pool_tiles + (p_last - lo) / KT + 1;
+  const int lead = a.keep_first < lo ? a.keep_first : lo, skip = lo - lead, v_last = p_last - skip;  // virtual key indices: see the head of this file
+  const int all_key_tiles = pool_tiles + v_last / KT + 1;
   int tile_lo = 0, n_key_tiles = all_key_tiles;
   if (a.splits > 1) {
     const int per = (all_key_tiles + a.splits - 1) / a.splits;
@@ -541,15 +558,15 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
     bf16* sv = sk + KT * PITCH;
     const int gt = tile_lo + it;
     const bool pooled = gt < pool_tiles;
-    const int j0 = pooled ? gt * KT : lo + (gt - pool_tiles) * KT, last = pooled ? nb_last - 1 : p_last;
+    const int j0 = (pooled ? gt : gt - pool_tiles) * KT, last = pooled ? nb_last - 1 : v_last;
     const int tpp = pooled ? a.pool_slots : a.tokens_per_page, shift = pooled ? pool_shift : page_shift;
     const size_t hr = pooled ? pool_head_rows : head_rows;
     const bf16* kpool = pooled ? a.kp_pages : a.k_pages;
     const bf16* vpool = pooled ? a.vp_pages : a.v_pages;
     constexpr int CH = D / 8;  // 16-byte chunks per row
     for (int e = tid; e < KT * CH; e += nthreads) {
-      const int jj = e / CH, c = e % CH, j = j0 + jj;
-      const bool ok = j <= last;
+      const int jj = e / CH, c = e % CH, v = j0 + jj, j = pooled || v < lead ? v : v + skip;
+      const bool ok = v <= last;
       const int pg = shift >= 0 ? (j >> shift) : j / tpp;
       const size_t row = ok ? hr + size_t(pages[pg]) * tpp + (j - pg * tpp) : 0;
       cp_async_16(sk + jj * PITCH + c * 8, kpool + row * D + c * 8, ok);
@@ -604,9 +621,9 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
       const bf16* sv = same_kv ? sk : sk + KT * PITCH;
       const int gt = tile_lo + it;
       const bool pooled = gt < pool_tiles;
-      const int j0 = pooled ? gt * KT : lo + (gt - pool_tiles) * KT;
+      const int j0 = (pooled ? gt : gt - pool_tiles) * KT;
       // a tile whose every key every row of the query tile sees (most tiles of a long window) needs no masks
-      const bool every_key_seen = pooled ? j0 + KT <= nb_first : (j0 + KT - 1 <= p0 && j0 >= lo_last);
+      const bool every_key_seen = pooled ? j0 + KT <= nb_first : (j0 < lead ? j0 + KT <= lead : j0 + skip + KT - 1 <= p0 && j0 + skip >= lo_last);
       float s[KT / 8][4];
 #pragma unroll
       for (int nb = 0; nb < KT / 8; ++nb) {
@@ -624,8 +641,8 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
         for (int e = 0; e < 4; ++e) {
           float sc = capped ? smax_softcap_scaled(s[nb][e], cap_mul, a.softcap) : s[nb][e] * a.scale;
           if (!every_key_seen || (sloped && !pooled)) {
-            const int j = j0 + nb * 8 + 2 * t + (e & 1), pi = (e & 2) ? pi1 : pi0;
-            const bool seen = pooled ? j < ((e & 2) ? nb1 : nb0) : (j <= pi && j >= ((e & 2) ? lo1 : lo0));
+            const int v = j0 + nb * 8 + 2 * t + (e & 1), j = pooled || v < lead ? v : v + skip, pi = (e & 2) ? pi1 : pi0;
+            const bool seen = pooled ? j < ((e & 2) ? nb1 : nb0) : (j <= pi && (j >= ((e & 2) ? lo1 : lo0) || j < a.keep_first));
             if (sloped && !pooled) sc -= slope * float(pi - j);
             sc = seen ? sc : -INFINITY;
           }
@@ -708,9 +725,16 @@ __global__ void __launch_bounds__(128) softmax_attention_mma_kernel(const Softma
     }
     return;
   }
-  const float f0 = a.out_scale / l_run[0] * (g < nr ? smax_gate(a.gate, a.ld_gate, r0 + g, h) : 1.0f);
-  const float f1 = a.out_scale / l_run[1] * (g + 8 < nr ? smax_gate(a.gate, a.ld_gate, r0 + g + 8, h) : 1.0f);
+  const float f0 = a.out_scale / l_run[0] * (g < nr ? smax_gate(a, r0 + g, h) : 1.0f);
+  const float f1 = a.out_scale / l_run[1] * (g + 8 < nr ? smax_gate(a, r0 + g + 8, h) : 1.0f);
   bf16* out0 = a.out + size_t(r0 + g) * a.ld_out + h * D + part * DVW + 2 * t;
+  if (a.value_gate) {
+#pragma unroll
+    for (int nb = 0; nb < NB; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (g + (e & 2) * 4 < nr) o[nb][e] *= smax_value_gate(a, r0 + g + (e & 2) * 4, h, part * DVW + nb * 8 + 2 * t + (e & 1));
+  }
   bf16* out1 = out0 + size_t(8) * a.ld_out;
 #pragma unroll
   for (int nb = 0; nb < NB; ++nb) {
@@ -757,7 +781,8 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
   const int nb = smax_blocks_seen(pos, a.window, a.pool), pool_tiles = (nb + KT - 1) / KT;
   const int pool_shift = (a.pool_slots & (a.pool_slots - 1)) == 0 && a.pool_slots > 0 ? __ffs(a.pool_slots) - 1 : -1;
   const size_t pool_head_rows = size_t(kvh) * a.num_pages * a.pool_slots;
-  const int all_key_tiles = pool_tiles + (pos - lo) / KT + 1;
+  const int lead = a.keep_first < lo ? a.keep_first : lo, skip = lo - lead, v_last = pos - skip;  // virtual key indices: see the head of this file
+  const int all_key_tiles = pool_tiles + v_last / KT + 1;
   const int per = (all_key_tiles + a.splits - 1) / a.splits;
   const int tile_lo = int(blockIdx.z) * per;
   int n_key_tiles = all_key_tiles - tile_lo < per ? all_key_tiles - tile_lo : per;
@@ -768,15 +793,15 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
     bf16* sv = sk + KT * PITCH;
     const int gt = tile_lo + it;
     const bool pooled = gt < pool_tiles;
-    const int j0 = pooled ? gt * KT : lo + (gt - pool_tiles) * KT, last = pooled ? nb - 1 : pos;
+    const int j0 = (pooled ? gt : gt - pool_tiles) * KT, last = pooled ? nb - 1 : v_last;
     const int tpp = pooled ? a.pool_slots : a.tokens_per_page, shift = pooled ? pool_shift : page_shift;
     const size_t hr = pooled ? pool_head_rows : head_rows;
     const bf16* kpool = pooled ? a.kp_pages : a.k_pages;
     const bf16* vpool = pooled ? a.vp_pages : a.v_pages;
     constexpr int CH = D / 8;
     for (int e = tid; e < KT * CH; e += NT) {
-      const int jj = e / CH, c = e % CH, j = j0 + jj;
-      const bool ok = j <= last;
+      const int jj = e / CH, c = e % CH, v = j0 + jj, j = pooled || v < lead ? v : v + skip;
+      const bool ok = v <= last;
       const int pg = shift >= 0 ? (j >> shift) : j / tpp;
       const size_t r = ok ? hr + size_t(pages[pg]) * tpp + (j - pg * tpp) : 0;
       cp_async_16(sk + jj * PITCH + c * 8, kpool + r * D + c * 8, ok);
@@ -825,8 +850,8 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
     const bf16* sv = same_kv ? sk : sk + KT * PITCH;
     const int gt = tile_lo + it;
     const bool pooled = gt < pool_tiles;
-    const int j0 = (pooled ? gt * KT : lo + (gt - pool_tiles) * KT) + warp * 16;  // this warp's 16 keys
-    if (j0 <= (pooled ? nb - 1 : pos)) {
+    const int j0 = (pooled ? gt : gt - pool_tiles) * KT + warp * 16;  // this warp's 16 keys
+    if (j0 <= (pooled ? nb - 1 : v_last)) {
       float c[4] = {0.0f, 0.0f, 0.0f, 0.0f};
       const bf16* k0 = sk + (warp * 16 + g) * PITCH + 2 * t;
 #pragma unroll
@@ -840,11 +865,11 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
       }
       // c[0], c[1]: key j0 + g, heads 2t, 2t + 1;  c[2], c[3]: key j0 + g + 8
       const int ja = j0 + g, jb = j0 + g + 8;
-      const bool sa_ = pooled ? ja < nb : ja <= pos;  // (no tile starts before the first visible key)
-      const bool sb_ = pooled ? jb < nb : jb <= pos;
+      const bool sa_ = ja <= (pooled ? nb - 1 : v_last);  // (every key of the walk up to its end is visible)
+      const bool sb_ = jb <= (pooled ? nb - 1 : v_last);
 #pragma unroll
       for (int e = 0; e < 4; ++e) c[e] = a.softcap > 0.0f ? smax_softcap_scaled(c[e], cap_mul, a.softcap) : c[e] * a.scale;
-      const float da = pooled ? 0.0f : float(pos - ja), db = pooled ? 0.0f : float(pos - jb);
+      const float da = pooled ? 0.0f : float(v_last - ja), db = pooled ? 0.0f : float(v_last - jb);  // (distances: slopes do not go with kept tokens)
       c[0] = sa_ ? c[0] - slope0 * da : -INFINITY;
       c[1] = sa_ ? c[1] - slope1 * da : -INFINITY;
       c[2] = sb_ ? c[2] - slope0 * db : -INFINITY;
@@ -930,7 +955,7 @@ __global__ void __launch_bounds__(kSdecWarps * 32) softmax_attention_decode_kern
         a.part_ml[base * 2 + 1] = L;
       }
     } else {
-      a.out[size_t(row) * a.ld_out + h * D + col] = __float2bfloat16_rn(acc * a.out_scale / L * smax_gate(a.gate, a.ld_gate, row, h));
+      a.out[size_t(row) * a.ld_out + h * D + col] = __float2bfloat16_rn(acc * a.out_scale / L * smax_gate(a, row, h) * smax_value_gate(a, row, h, col));
     }
   }
 }
@@ -948,7 +973,7 @@ __global__ void __launch_bounds__(128) softmax_attention_merge_kernel(const Soft
     const float* ml = a.part_ml + ((size_t(z) * a.rows + row) * a.heads + h) * 2;
     if (ml[0] != -INFINITY) L += __expf(ml[0] - M) * ml[1];
   }
-  const float gate = smax_gate(a.gate, a.ld_gate, row, h);
+  const float gate = smax_gate(a, row, h);
   for (int c = lane; c < D; c += 32) {
     float acc = 0.0f;
     for (int z = 0; z < a.splits; ++z) {
@@ -956,7 +981,7 @@ __global__ void __launch_bounds__(128) softmax_attention_merge_kernel(const Soft
       const float mz = a.part_ml[base * 2];
       if (mz != -INFINITY) acc = fmaf(__expf(mz - M), a.part_o[base * D + c], acc);
     }
-    a.out[size_t(row) * a.ld_out + h * D + c] = __float2bfloat16_rn(acc * a.out_scale / L * gate);
+    a.out[size_t(row) * a.ld_out + h * D + c] = __float2bfloat16_rn(acc * a.out_scale / L * gate * smax_value_gate(a, row, h, c));
   }
 }
 

@@ -28,9 +28,11 @@ from . import params as params_lib
 from .maxengine import ExistingPrefix, MaxEngine, ResultTokens  # noqa: F401  (same result types)
 
 _MIXERS = {"window_sigmoid": _lib.MIXER_WINDOW_SIGMOID, "composite": _lib.MIXER_COMPOSITE}
-_NORMS = {"out_gain": _lib.NORM_OUT_GAIN, "sandwich": _lib.NORM_SANDWICH, "parallel": _lib.NORM_PARALLEL, "pre": _lib.NORM_PRE}
-_FF_KINDS = {"none": _lib.FF_GELU_GATED, "gelu": _lib.FF_GELU_GATED, "clamped": _lib.FF_CLAMPED_GATED, "moe": _lib.FF_MOE, "relu2": _lib.FF_RELU2}
-_RECURRENCES = {"gla": _lib.REC_GLA, "mlstm": _lib.REC_MLSTM, "delta": _lib.REC_DELTA, "gdelta": _lib.REC_GDELTA}
+_NORMS = {"out_gain": _lib.NORM_OUT_GAIN, "sandwich": _lib.NORM_SANDWICH, "parallel": _lib.NORM_PARALLEL, "pre": _lib.NORM_PRE,
+          "out_layer": _lib.NORM_OUT_LAYER}
+_FF_KINDS = {"none": _lib.FF_GELU_GATED, "gelu": _lib.FF_GELU_GATED, "clamped": _lib.FF_CLAMPED_GATED, "moe": _lib.FF_MOE, "relu2": _lib.FF_RELU2,
+             "gelu_up": _lib.FF_GELU}
+_RECURRENCES = {"gla": _lib.REC_GLA, "mlstm": _lib.REC_MLSTM, "delta": _lib.REC_DELTA, "gdelta": _lib.REC_GDELTA, "decay": _lib.REC_DECAY}
 QUERY_TILE_ROWS = 16  # rows of one query tile of the attention kernels (csrc/window_attention_mma.cuh, csrc/softmax_attention.cuh)
 
 _LAYER_MATS = ("wqkv", "wo", "w_gate_up", "w_down", "w_in")
@@ -39,7 +41,7 @@ _LAYER_VECS = ("bqkv", "q_norm", "k_norm", "dist_bias", "head_bias", "talk", "no
 _ATTN_VECS = ("q_norm", "k_norm", "slopes", "sink", "temp", "talk")
 _LATENT_MATS = ("w_uq", "w_uk_t", "w_uv")
 _LATENT_VECS = ("q_norm", "kv_norm", "sink")
-_REC_VECS = ("decay_up_t", "decay_bias", "gate_bias", "out_norm", "conv_w", "a_log")
+_REC_VECS = ("decay_up_t", "decay_bias", "gate_bias", "out_norm", "conv_w", "a_log", "head_decay")
 _REC_MATS = ("w_gate_up", "decay_up2")
 _SIDE_MATS = ("gate", "proj")
 _SIDE_VECS = ("norm",)
@@ -69,6 +71,10 @@ def design_module(config):
     from . import fibelix
 
     return fibelix
+  if config.decoder_block == "zakelorn":
+    from . import zakelorn
+
+    return zakelorn
   raise ValueError(f"decoder_block={config.decoder_block!r} is not a layered design")
 
 
@@ -109,7 +115,7 @@ class LayeredParams:
 
     self.embedding, self.head = mat(plan["embedding"]), mat(plan["head"])
     self.final_gain, self.embed_scale = float(plan["final_gain"]), float(plan["embed_scale"])
-    self.final_norm = vec(plan.get("final_norm"))
+    self.final_norm, self.final_norm_b = vec(plan.get("final_norm")), vec(plan.get("final_norm_b"))
     self.logit_softcap = float(plan.get("logit_softcap") or 0.0)
     self.logit_scale = float(plan.get("logit_scale") or 1.0)
     self.norm_groups = int(plan.get("norm_groups") or 0)
@@ -268,7 +274,7 @@ class LayeredEngine(MaxEngine):
             Gv, maps, dk = int(a["kv_heads"]), max(1, int(a.get("maps") or 1)), int(a["dim"])
             Gk, dk = (1, Gv * dk) if a.get("talk") is not None else (Gv * maps, dk)
             kp, vp = pools(Gk, dk, Gv, int(a["vdim"]))
-          for k in ("heads", "kv_heads", "dim", "vdim", "window", "rot_dims", "values_are_keys", "rot_half", "shared_kv", "head_gate", "chunk", "maps"):
+          for k in ("heads", "kv_heads", "dim", "vdim", "window", "rot_dims", "values_are_keys", "rot_half", "shared_kv", "head_gate", "chunk", "maps", "keep_first", "value_gate"):
             setattr(d.attn, k, int(a.get(k, 0)))
           d.attn.diff_lambda, d.attn.diff_scale = float(a.get("diff_lambda", 0.0)), float(a.get("diff_scale", 0.0))
           d.attn.scale, d.attn.out_scale = float(a["scale"]), float(a["out_scale"])
@@ -310,6 +316,7 @@ class LayeredEngine(MaxEngine):
           d.rec.decay_rate, d.rec.key_eps = float(r.get("decay_rate", 0.0)), float(r.get("key_eps", 0.0))
           for k in ("decay_up_t", "decay_bias", "gate_bias", "out_norm"):
             setattr(d.rec, k, ptr(r.get(k)))
+          d.rec.head_decay, d.rec.norm_whole = ptr(r.get("head_decay")), int(r.get("norm_whole", 0))
           H, dk, dv = int(r["heads"]), int(r["dim"]), int(r["vdim"])
           f32 = torch.float32
           if r["kind"] == "gdelta":
@@ -332,7 +339,7 @@ class LayeredEngine(MaxEngine):
           d.moe.limit, d.moe.shared_limit = float(m["limit"]), float(m["shared_limit"])
           for k in ("w_router", "correction", "router_bias", "w_gate_up", "w_down", "shared_gate_up", "shared_down"):
             setattr(d.moe, k, ptr(m.get(k)))
-          for k in ("score_softmax", "plain_weights", "act_silu", "chosen_softmax"):
+          for k in ("score_softmax", "plain_weights", "act_silu", "chosen_softmax", "groups_max", "identity", "shared_gate"):
             setattr(d.moe, k, int(m.get(k, 0)))
         sd = l.get("side")
         if sd:
@@ -354,7 +361,8 @@ class LayeredEngine(MaxEngine):
         tokens_per_page=pm.tokens_per_page, max_pages_per_group=pm.max_pages_per_group, eps=float(cfg.normalization_layer_epsilon),
         embed_scale=lp.embed_scale, final_gain=lp.final_gain, embedding=lp.embedding.data_ptr(), head=lp.head.data_ptr(),
         final_norm=ptr(lp.final_norm), logit_softcap=lp.logit_softcap, norm_groups=lp.norm_groups, logit_scale=lp.logit_scale,
-        embed_norm=ptr(lp.embed_norm), side_embed=ptr(lp.side_embed), side_width=int(lp.side_embed.shape[1]) if lp.side_embed is not None else 0)
+        embed_norm=ptr(lp.embed_norm), side_embed=ptr(lp.side_embed), side_width=int(lp.side_embed.shape[1]) if lp.side_embed is not None else 0,
+        final_norm_b=ptr(lp.final_norm_b))
     _lib.check(self.lib.mtx_layered_create(ctypes.byref(c), descs, ctypes.byref(self._handle)))
     ws = int(self.lib.mtx_layered_workspace_bytes(self._handle))
     self._ws = torch.empty(ws + 1024, dtype=torch.uint8, device=dev)

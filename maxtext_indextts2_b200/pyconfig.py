@@ -36,8 +36,9 @@ _VALID_SAMPLING = ("greedy", "weighted", "nucleus", "topk")
 _VALID_AXIS_ORDER = ("0,1,2,3", "0,2,1,3")
 # Designs whose layers are listed one by one (`layer_specs`) and run on the layered engine (layered_engine.py), keyed by
 # decoder_block; ARCHITECTURES maps the "architecture" of a model folder's config.json to the block.
-LAYERED_BLOCKS = ("kifusun", "gugidra", "ginodra", "ligidra", "fibelix")
-ARCHITECTURES = {"Kifusun": "kifusun", "Gugidra": "gugidra", "Ginodra": "ginodra", "Ligidra": "ligidra", "Fibelix": "fibelix"}
+LAYERED_BLOCKS = ("kifusun", "gugidra", "ginodra", "ligidra", "fibelix", "zakelorn")
+ARCHITECTURES = {"Kifusun": "kifusun", "Gugidra": "gugidra", "Ginodra": "ginodra", "Ligidra": "ligidra", "Fibelix": "fibelix",
+                 "Zakelorn": "zakelorn"}
 
 
 def _string_to_bool(s: str) -> bool:
@@ -146,6 +147,10 @@ def _validate_layered(keys: dict) -> None:
     from . import fibelix
 
     fibelix.validate_layer_specs(keys["layer_specs"])
+  if keys["decoder_block"] == "zakelorn":
+    from . import zakelorn
+
+    zakelorn.validate_layer_specs(keys["layer_specs"])
 
 
 def _validate(keys: dict) -> None:
@@ -322,6 +327,10 @@ def from_model_dict(model: dict, **overrides) -> HyperParameters:
     from . import fibelix
 
     keys = fibelix.config_keys(model)
+  elif block == "zakelorn":
+    from . import zakelorn
+
+    keys = zakelorn.config_keys(model)
   keys.update(decoder_block=block, attention="paged", scan_layers=False, weight_dtype="bfloat16")
   keys.update(overrides)
   if "max_prefill_predict_length" not in overrides:  # any prompt that fits the sequence
