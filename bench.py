@@ -66,7 +66,7 @@ def parse_args():
   ap.add_argument("--no-verify", action="store_true", help="skip the oracle check of one step of the timed state")
   ap.add_argument("--prompt-len", type=int, default=4000, help="--mode prefill: prompt tokens (BASELINE configs[3]: 4000 of P = 4096)")
   ap.add_argument("--size", default="all", help="--mode layered: one of the sizes of LAYERED_SIZES, or all")
-  ap.add_argument("--design", default="kifusun", choices=["kifusun", "gugidra", "ginodra", "ligidra", "fibelix"], help="--mode layered: the layered design that is measured beside gemma3")
+  ap.add_argument("--design", default="kifusun", choices=["kifusun", "gugidra", "ginodra", "ligidra", "fibelix", "zakelorn"], help="--mode layered: the layered design that is measured beside gemma3")
   ap.add_argument("--mode", default="batch", choices=["batch", "vocab-parallel", "prefill", "layered"],
                   help="batch: request-batch partitioned, no collective (default); vocab-parallel: every GPU decodes the same --batch slots, "
                        "the logits projection is sharded over the GPUs and one NCCL all-gather carries the per-shard candidates")
@@ -614,7 +614,7 @@ def run_layered(args):
   """--mode layered: prefill and decode throughput of a layered design (--design) on the layered engine beside the gemma3 block
   (the closest existing model: softmax attention with rotary positions and grouped key heads, norms before and after every
   sublayer, gated feed-forward) at equal layer sizes, both through MaxEngine.  One JSON line per size."""
-  from maxtext_indextts2_b200 import fibelix, ginodra, gugidra, kifusun, ligidra, maxengine, pyconfig
+  from maxtext_indextts2_b200 import fibelix, ginodra, gugidra, kifusun, ligidra, maxengine, pyconfig, zakelorn
 
   D = args.design  # (the keys of the output line carry the design's name)
   names = list(LAYERED_SIZES) if args.size == "all" else [args.size]
@@ -674,6 +674,17 @@ def run_layered(args):
       model = fibelix.model_dict(z["width"], z["vocab"], layers)
       ctx = (C // (2 * W) * 2 + 1) * W
       T = max(T, ctx + 64)
+    elif D == "zakelorn":
+      # Zakelorn at the same sizes: in every layer an attention with gemma3's heads and window (four kept first tokens, half of every
+      # head's channels rotated) beside a lightning attention of as many value channels (heads of 64 or 128); dense feed-forwards of
+      # gemma3's active size (two matrices of 3/2 ff) in turn with routed ones (16 experts of ff / 8 and 4 identity experts in 4 groups, four
+      # choices per token, a shared expert of ff / 2)
+      H, G, d, F, W = z["heads"], z["kv_heads"], z["dim"], z["ff"], z["window"]
+      dr = min(d, 128)
+      ffs = [zakelorn.dense_ff(F * 3 // 2), zakelorn.moe_ff(16, 4, F // 8, identity=4, groups=4, keep=3, shared_ff=F // 2)]
+      layers = [zakelorn.parallel_layer(zakelorn.attention_part(H, G, d, window=W, keep_first=4, rot_dims=d // 2), zakelorn.lightning_part(H * d // dr, dr),
+                                        0.8, 1.1, ffs[i % 2]) for i in range(L)]
+      model = zakelorn.model_dict(z["width"], z["vocab"], layers, embed_scale=z["width"] ** 0.5)
     else:
       # Gugidra at the same sizes: attention + mLSTM layers and GLA layers in turn; the attention has gemma3's heads (no window: the
       # design has none), the recurrences half as many key channels per head; dense feed-forwards of gemma3's size in turn with
