@@ -2,7 +2,8 @@
 // batches whose keys and values live in page pools.  Host code only: the kernels are in linear_any.cuh (any-shape projections, also
 // grouped by expert), gemm_rows.cuh (the tcgen05 projections, for shapes made of whole 128 x 64 tiles), layer_ops.cuh (norms,
 // residual, cache append), grouped_gemm.cuh (the experts' products of steps with many rows), window_attention*.cuh (the sigmoid window mixer), softmax_attention.cuh (causal softmax attention with
-// rotary positions), multi_attention.cuh (its tensor-core kernels for two score maps per head and for scores mixed over the heads), recurrent_mixers.cuh (GLA, mLSTM and the delta rule over state slots), latent_attention.cuh (attention through
+// rotary positions), multi_attention.cuh (its tensor-core kernels for two score maps per head and for scores mixed over the heads), recurrent_mixers.cuh (GLA, mLSTM, the delta rule and decayed sums over state slots), decayed_sums.cuh (decayed sums of prompt portions on the
+// tensor cores), latent_attention.cuh (attention through
 // cached latents) and moe.cuh (routing).
 #include <cmath>
 #include <cstdio>
@@ -19,6 +20,7 @@
 #include "softmax_attention.cuh"
 #include "multi_attention.cuh"
 #include "recurrent_mixers.cuh"
+#include "decayed_sums.cuh"
 #include "latent_attention.cuh"
 #include "moe.cuh"
 #include "host_util.cuh"
@@ -144,8 +146,9 @@ __global__ void gate_up_bf16_kernel(const bf16* src, bf16* act, int ff, long lon
   }
 }
 
-// eight columns per thread: fp32 values of a bf16 projection, the columns [silu0, silu1) through silu and rounded to bf16 again
-__global__ void __launch_bounds__(256) bf16_cols_to_f32_kernel(const bf16* src, float* dst, int n, int silu0, int silu1, long long groups) {
+// eight columns per thread: fp32 values of a bf16 projection, the columns [silu0, silu1) through silu and rounded to bf16 again, or (in_place:
+// silu0 and silu1 multiples of 8) these columns through silu where they are, for a reader of bf16
+__global__ void __launch_bounds__(256) bf16_cols_to_f32_kernel(bf16* src, float* dst, int n, int silu0, int silu1, int in_place, long long groups) {
   griddep_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < groups; i += (long long)gridDim.x * blockDim.x) {
     const uint4 q = *reinterpret_cast<const uint4*>(src + i * 8);
@@ -162,6 +165,10 @@ __global__ void __launch_bounds__(256) bf16_cols_to_f32_kernel(const bf16* src, 
 #pragma unroll
       for (int e = 0; e < 8; ++e)
         if (c0 + e >= silu0 && c0 + e < silu1) v[e] = __bfloat162float(__float2bfloat16_rn(silu_gate_f(v[e], 1.0f)));
+      if (in_place) {
+        *reinterpret_cast<uint4*>(src + i * 8) = make_uint4(smax_pack_bf16(v[0], v[1]), smax_pack_bf16(v[2], v[3]), smax_pack_bf16(v[4], v[5]), smax_pack_bf16(v[6], v[7]));
+        continue;
+      }
     }
     *reinterpret_cast<float4*>(dst + i * 8) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(dst + i * 8 + 4) = make_float4(v[4], v[5], v[6], v[7]);
@@ -251,7 +258,7 @@ int run_linear_umma(mtx_layered* e, const void* a, const void* w, const float* b
   const int blocks = int((total + 255) / 256 < 148 * 8 ? (total + 255) / 256 : 148 * 8);
   const long long groups = total / 8;  // (n is a multiple of 128)
   const int blocks8 = int((groups + 255) / 256 < 148 * 8 ? (groups + 255) / 256 : 148 * 8);
-  if (EPI == LIN_SILU_COLS) return launch(bf16_cols_to_f32_kernel, dim3(blocks8), dim3(256), 0, st, tmp, out, n, silu0, silu1, groups);
+  if (EPI == LIN_SILU_COLS) return launch(bf16_cols_to_f32_kernel, dim3(blocks8), dim3(256), 0, st, static_cast<bf16*>(e->obf), out, n, silu0, silu1, 0, groups);
   if (EPI == LIN_ACT || EPI == LIN_RELU2 || EPI == LIN_GELU) {
     if (ldo <= 0) ldo = n;
     if (ldo % 8 == 0 && (reinterpret_cast<uintptr_t>(act) & 15) == 0) return launch(act8_bf16_kernel, dim3(blocks8), dim3(256), 0, st, tmp, static_cast<bf16*>(act), n, ldo, groups, EPI);
@@ -1701,6 +1708,30 @@ int project_out_layer_norm(mtx_layered* e, const void* a, const void* w, int k, 
   return out_layer_norm<T>(e, oa, nw, nb, rows, st);
 }
 
+template <typename SRC, int MT>
+int launch_decayed_chunks_t(const DecayedChunksArgs& da, int n_runs, cudaStream_t st) {
+  const size_t smem = decayed_chunks_smem_bytes(da.dim);
+  static size_t have = 0;  // per instantiation
+  if (smem > 48 * 1024 && smem > have) {
+    MTX_CUDA(cudaFuncSetAttribute(decayed_chunks_kernel<SRC, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    have = smem;
+  }
+  return launch(decayed_chunks_kernel<SRC, MT>, dim3(n_runs, da.heads, (da.vdim + kDcCols - 1) / kDcCols), dim3(kDcThreads), smem, st, da);
+}
+
+template <typename SRC>
+int launch_decayed_chunks(const DecayedChunksArgs& da, int n_runs, cudaStream_t st) {
+  if (da.dim <= 64) return launch_decayed_chunks_t<SRC, 1>(da, n_runs, st);
+  if (da.dim <= 128) return launch_decayed_chunks_t<SRC, 2>(da, n_runs, st);
+  return launch_decayed_chunks_t<SRC, 4>(da, n_runs, st);
+}
+
+// decayed sums in chunks: bf16 engines, steps whose runs are several tokens long on average (else the token walk)
+bool use_decayed_chunks(const mtx_layered* e, const mtx_ragged_batch& b) {
+  static int on = env_int("MTX_DECAY_CHUNKS", 1);
+  return on != 0 && !e->cfg.float32 && b.rows >= 4 * b.n_runs;
+}
+
 // a MTX_NORM_OUT_LAYER layer: both sublayers read x itself (xa = x in the matmul dtype)
 template <typename T>
 int outlayer_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream_t st) {
@@ -1712,8 +1743,15 @@ int outlayer_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
   const CompositeCols cc = composite_cols(l);
   const mtx_softmax_attn_desc& a = l.attn;
   const mtx_recurrent_desc& r = l.rec;
+  const bool chunks = r.kind != 0 && use_decayed_chunks(e, b);
+  const bool chunks_bf16 = chunks && takes_umma(e, rows, n_in, E) && cc.rq % 8 == 0 && cc.rg % 8 == 0;  // they read the projection where the GEMM left it
   // (the recurrence's q, k and v are next to one another: silu on the way)
-  MTX_TRY((linear<T, LIN_SILU_COLS>(e, xa, l.w_in, nullptr, e->qkv, nullptr, rows, n_in, E, st, 0.0f, 0, cc.rq, r.kind != 0 ? cc.rg : cc.rq)));
+  if (chunks_bf16) {
+    MTX_TRY(run_umma_raw(e, xa, l.w_in, rows, n_in, E, st));
+    const long long groups = (long long)rows * n_in / 8;
+    const int blocks = int((groups + 255) / 256 < 148 * 8 ? (groups + 255) / 256 : 148 * 8);
+    MTX_TRY(launch(bf16_cols_to_f32_kernel, dim3(blocks), dim3(256), 0, st, static_cast<bf16*>(e->obf), e->qkv, n_in, cc.rq, cc.rg, 1, groups));
+  } else MTX_TRY((linear<T, LIN_SILU_COLS>(e, xa, l.w_in, nullptr, e->qkv, nullptr, rows, n_in, E, st, 0.0f, 0, cc.rq, r.kind != 0 ? cc.rg : cc.rq)));
   if (a.heads > 0) {
     QkPrepareArgs<T> qa;
     memset(&qa, 0, sizeof(qa));
@@ -1763,25 +1801,48 @@ int outlayer_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
     MTX_TRY(run_softmax_attention<T>(e, sa, b, st));
   }
   if (r.kind != 0) {
-    RecScanArgs ra;
-    memset(&ra, 0, sizeof(ra));
-    ra.proj = e->qkv;
-    ra.ld = n_in;
-    ra.q_col = cc.rq;
-    ra.k_col = cc.rk;
-    ra.v_col = cc.rv;
-    ra.o = e->rec_o;
-    ra.state_s = r.state_s;
-    ra.head_decay = r.head_decay;
-    ra.run_row0 = b.run_row0;
-    ra.group = b.group;
-    ra.pos = b.pos;
-    ra.heads = r.heads;
-    ra.dim = r.dim;
-    ra.vdim = r.vdim;
-    ra.q_scale = r.q_scale;
-    ra.vec4 = (n_in % 4 == 0 && cc.rq % 4 == 0 && r.dim % 4 == 0 && r.vdim % 4 == 0) ? 1 : 0;
-    MTX_TRY(launch_rec_scan<REC_DECAY>(e, ra, b.n_runs, rows, st));
+    if (chunks) {
+      DecayedChunksArgs da;
+      memset(&da, 0, sizeof(da));
+      da.src = chunks_bf16 ? e->obf : static_cast<const void*>(e->qkv);
+      da.ld = n_in;
+      da.q_col = cc.rq;
+      da.k_col = cc.rk;
+      da.v_col = cc.rv;
+      da.o = e->rec_o;
+      da.state = r.state_s;
+      da.head_decay = r.head_decay;
+      da.run_row0 = b.run_row0;
+      da.group = b.group;
+      da.pos = b.pos;
+      da.heads = r.heads;
+      da.dim = r.dim;
+      da.vdim = r.vdim;
+      da.q_scale = r.q_scale;
+      da.vec8 = (n_in % 8 == 0 && cc.rq % 8 == 0 && r.dim % 8 == 0 && r.vdim % 8 == 0) ? 1 : 0;
+      if (chunks_bf16) MTX_TRY(launch_decayed_chunks<bf16>(da, b.n_runs, st));
+      else MTX_TRY(launch_decayed_chunks<float>(da, b.n_runs, st));
+    } else {
+      RecScanArgs ra;
+      memset(&ra, 0, sizeof(ra));
+      ra.proj = e->qkv;
+      ra.ld = n_in;
+      ra.q_col = cc.rq;
+      ra.k_col = cc.rk;
+      ra.v_col = cc.rv;
+      ra.o = e->rec_o;
+      ra.state_s = r.state_s;
+      ra.head_decay = r.head_decay;
+      ra.run_row0 = b.run_row0;
+      ra.group = b.group;
+      ra.pos = b.pos;
+      ra.heads = r.heads;
+      ra.dim = r.dim;
+      ra.vdim = r.vdim;
+      ra.q_scale = r.q_scale;
+      ra.vec4 = (n_in % 4 == 0 && cc.rq % 4 == 0 && r.dim % 4 == 0 && r.vdim % 4 == 0) ? 1 : 0;
+      MTX_TRY(launch_rec_scan<REC_DECAY>(e, ra, b.n_runs, rows, st));
+    }
     RecOutArgs<T> oa;
     memset(&oa, 0, sizeof(oa));
     oa.o = e->rec_o;

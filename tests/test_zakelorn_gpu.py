@@ -365,6 +365,20 @@ def test_a_slot_that_is_taken_again_starts_from_an_empty_state():
   assert rel_err(in_portions(engine, b, [], slot=0, decode=12), ref.forward(cfg, t, b)) < TIGHT
 
 
+@pytest.mark.parametrize("dim,vdim", [(8, 8), (64, 24), (128, 128), (200, 40), (10, 7)])
+def test_decayed_sums_in_chunks_and_token_by_token(dim, vdim):
+  """bf16 engines: portions take the chunked kernel, single tokens the token walk, both from the same state; decays that keep
+  everything, forget everything and anything between, portions that end before, at and after a chunk's edge."""
+  cfg = model([par(right=lin(heads=5, dim=dim, vdim=vdim, decay=[1.0, 0.0, 0.999, 0.3, 0.9]), left_scale=0.0)], width=64)
+  toks = tokens_for(cfg, 300)
+  t = weights(cfg, 8)
+  want = ref.forward(cfg, t, toks)
+  engine = make_engine(cfg, t, dtype="bfloat16", tokens_per_page=16, num_pages=60, max_len=320)
+  assert rms_err(whole(engine, toks), want) < LOOSE / 2
+  for cuts, decode in (([63, 65, 64, 4], 5), ([128, 1, 129], 3), ([5, 59, 2, 190], 9), ([], 300)):
+    assert rms_err(in_portions(engine, toks, cuts, decode=decode), want[: sum(cuts) + decode]) < LOOSE / 2, cuts
+
+
 # ---- other sizes ------------------------------------------------------------------------------------------------------------------
 
 SIZES = {
