@@ -1856,10 +1856,12 @@ int outlayer_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
     oa.heads = r.heads;
     oa.vdim = r.vdim;
     oa.gate_silu = r.gate_silu;
-    oa.norm_whole = r.norm_whole;
     oa.eps = c.eps;
     oa.out_scale = r.out_scale;
-    MTX_TRY(launch(recurrent_out_kernel<T>, dim3(rows), dim3(256), 0, st, oa));
+    const bool vec = (r.heads * r.vdim) % 4 == 0 && n_in % 4 == 0 && cc.rg % 4 == 0 && cc.k_out % 4 == 0 && cc.out_rec % 4 == 0;
+    if (!r.norm_whole) MTX_TRY(launch(recurrent_out_kernel<T>, dim3(rows), dim3(256), 0, st, oa));
+    else if (vec) MTX_TRY(launch(recurrent_out_whole_kernel<T, 4>, dim3(rows), dim3(256), 0, st, oa));
+    else MTX_TRY(launch(recurrent_out_whole_kernel<T, 1>, dim3(rows), dim3(256), 0, st, oa));
   }
   MTX_TRY(project_out_layer_norm<T>(e, mix, l.wo, cc.k_out, l.norm1, l.norm1b, rows, st));
   if (l.ff_kind == MTX_FF_MOE) {
@@ -2166,6 +2168,7 @@ int check_outlayer(mtx_layered* e, int i) {
     if (r.kind != MTX_REC_DECAY) return fail(MTX_ERR_UNSUPPORTED, "layer %d: the recurrence beside layer norms on the outputs is the decayed sum", i);
     if (r.heads < 1 || r.dim < 1 || r.vdim < 1 || r.dim > kRecSlices * 32) return fail(MTX_ERR_UNSUPPORTED, "layer %d: recurrence heads / dim (<= %d) / vdim", i, kRecSlices * 32);
     if (!r.state_s || !r.out_norm || !r.head_decay) return fail(MTX_ERR_ARG, "layer %d: the recurrence's state, output norm or decays are missing", i);
+    if (r.norm_whole && r.heads * r.vdim > 256 * kRecOutVec) return fail(MTX_ERR_UNSUPPORTED, "layer %d: heads * vdim = %d exceeds %d", i, r.heads * r.vdim, 256 * kRecOutVec);
     if (r.heads * r.vdim > e->max_rec_o) e->max_rec_o = r.heads * r.vdim;
   }
   const CompositeCols cc = composite_cols(l);

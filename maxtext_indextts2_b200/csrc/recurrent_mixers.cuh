@@ -23,7 +23,7 @@
 //   lowrank_split_kernel       the inputs of the gated delta rule's low-rank decay and gate projections in the matmul dtype
 //   gdelta_prepare_kernel      per row: the gated delta rule's convolutions, silu, unit vectors, decays and write strengths
 //   recurrent_scan_kernel      the walk
-//   recurrent_out_kernel<T>    per row and head (or over all heads of the row together): o / rms(o) * weight * gate(g) * out_scale -> the activation of the output projection
+//   recurrent_out_kernel<T>    per row and head (recurrent_out_whole_kernel: over all heads of the row together): o / rms(o) * weight * gate(g) * out_scale -> the activation of the output projection
 #pragma once
 
 #include "common.cuh"
@@ -643,7 +643,6 @@ struct RecOutArgs {
   int out_col;
   int heads, vdim, gate_silu;
   float eps, out_scale;
-  int norm_whole;       // 1: one root mean square over all heads of the row
 };
 
 // one CTA per row, a warp per head
@@ -651,20 +650,6 @@ template <typename T>
 __global__ void __launch_bounds__(256) recurrent_out_kernel(const RecOutArgs<T> a) {
   griddep_wait();
   const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, dv = a.vdim;
-  if (a.norm_whole) {
-    __shared__ float red[8];
-    const int n = a.heads * dv;
-    const float* o = a.o + size_t(r) * n;
-    const float* gate = a.proj + size_t(r) * a.ld + a.g_col;
-    float ss = 0.0f;
-    for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(o[c], o[c], ss);
-    const float inv = a.out_scale / sqrtf(block_sum(ss, red) / float(n) + a.eps);
-    for (int c = threadIdx.x; c < n; c += blockDim.x) {
-      const float g = gate[c], sig = 1.0f / (1.0f + expf(-g));
-      a.out[size_t(r) * a.ld_out + a.out_col + c] = to_act<T>(o[c] * inv * a.weight[c] * (a.gate_silu ? g * sig : sig));
-    }
-    return;
-  }
   for (int h = warp; h < a.heads; h += nw) {
     const float* o = a.o + size_t(r) * a.heads * dv + h * dv;
     float ss = 0.0f;
@@ -676,6 +661,58 @@ __global__ void __launch_bounds__(256) recurrent_out_kernel(const RecOutArgs<T> 
       const float sig = 1.0f / (1.0f + expf(-g));
       const float gate = a.gate_silu ? g * sig : sig;
       a.out[size_t(r) * a.ld_out + a.out_col + h * dv + c] = to_act<T>(o[c] * inv * a.weight[h * dv + c] * gate * a.out_scale);
+    }
+  }
+}
+
+// the same with ONE root mean square over all heads of the row (n = heads * vdim <= 256 * kRecOutVec).  The row and its gates stay in
+// registers across the reduction; V = 4: four channels per load (n, ld, ld_out, out_col and g_col multiples of 4), V = 1: any size
+constexpr int kRecOutVec = 32;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) recurrent_out_whole_kernel(const RecOutArgs<T> a) {
+  __shared__ float red[8];
+  constexpr int N = kRecOutVec / V;
+  griddep_wait();
+  const int r = blockIdx.x, n = a.heads * a.vdim;
+  const float* o = a.o + size_t(r) * n;
+  const float* gate = a.proj + size_t(r) * a.ld + a.g_col;
+  T* out = a.out + size_t(r) * a.ld_out + a.out_col;
+  float ov[N][V], gv[N][V], ss = 0.0f;
+#pragma unroll
+  for (int u = 0; u < N; ++u) {
+    const int c = (threadIdx.x + u * 256) * V;
+    if (c < n) {
+      if constexpr (V == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(o + c), y = *reinterpret_cast<const float4*>(gate + c);
+        ov[u][0] = x.x, ov[u][1] = x.y, ov[u][2] = x.z, ov[u][3] = x.w;
+        gv[u][0] = y.x, gv[u][1] = y.y, gv[u][2] = y.z, gv[u][3] = y.w;
+      } else {
+        ov[u][0] = o[c];
+        gv[u][0] = gate[c];
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(ov[u][e], ov[u][e], ss);
+    }
+  }
+  const float inv = a.out_scale / sqrtf(block_sum(ss, red) / float(n) + a.eps);
+#pragma unroll
+  for (int u = 0; u < N; ++u) {
+    const int c = (threadIdx.x + u * 256) * V;
+    if (c < n) {
+      float v[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float sig = 1.0f / (1.0f + expf(-gv[u][e]));
+        v[e] = ov[u][e] * inv * a.weight[c + e] * (a.gate_silu ? gv[u][e] * sig : sig);
+      }
+      if constexpr (V == 4 && sizeof(T) == 2) {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(out + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) out[c + e] = to_act<T>(v[e]);
+      }
     }
   }
 }
