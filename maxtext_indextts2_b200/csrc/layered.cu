@@ -1860,8 +1860,9 @@ int outlayer_layer(mtx_layered* e, int li, const mtx_ragged_batch& b, cudaStream
     oa.out_scale = r.out_scale;
     const bool vec = (r.heads * r.vdim) % 4 == 0 && n_in % 4 == 0 && cc.rg % 4 == 0 && cc.k_out % 4 == 0 && cc.out_rec % 4 == 0;
     if (!r.norm_whole) MTX_TRY(launch(recurrent_out_kernel<T>, dim3(rows), dim3(256), 0, st, oa));
-    else if (vec) MTX_TRY(launch(recurrent_out_whole_kernel<T, 4>, dim3(rows), dim3(256), 0, st, oa));
-    else MTX_TRY(launch(recurrent_out_whole_kernel<T, 1>, dim3(rows), dim3(256), 0, st, oa));
+    else if (vec && r.heads * r.vdim <= 256 * 8) MTX_TRY(launch(recurrent_out_whole_kernel<T, 4, 8>, dim3(rows), dim3(256), 0, st, oa));
+    else if (vec) MTX_TRY(launch(recurrent_out_whole_kernel<T, 4, kRecOutVec>, dim3(rows), dim3(256), 0, st, oa));
+    else MTX_TRY(launch(recurrent_out_whole_kernel<T, 1, kRecOutVec>, dim3(rows), dim3(256), 0, st, oa));
   }
   MTX_TRY(project_out_layer_norm<T>(e, mix, l.wo, cc.k_out, l.norm1, l.norm1b, rows, st));
   if (l.ff_kind == MTX_FF_MOE) {

@@ -666,13 +666,13 @@ __global__ void __launch_bounds__(256) recurrent_out_kernel(const RecOutArgs<T> 
 }
 
 // the same with ONE root mean square over all heads of the row (n = heads * vdim <= 256 * kRecOutVec).  The row and its gates stay in
-// registers across the reduction; V = 4: four channels per load (n, ld, ld_out, out_col and g_col multiples of 4), V = 1: any size
+// registers across the reduction (MAX channels per thread: 8, n <= 2048, or kRecOutVec); V = 4: four channels per load (n, ld, ld_out, out_col and g_col multiples of 4), V = 1: any size
 constexpr int kRecOutVec = 32;
 
-template <typename T, int V>
+template <typename T, int V, int MAX>
 __global__ void __launch_bounds__(256) recurrent_out_whole_kernel(const RecOutArgs<T> a) {
   __shared__ float red[8];
-  constexpr int N = kRecOutVec / V;
+  constexpr int N = MAX / V;
   griddep_wait();
   const int r = blockIdx.x, n = a.heads * a.vdim;
   const float* o = a.o + size_t(r) * n;
